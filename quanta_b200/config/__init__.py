@@ -1,5 +1,6 @@
 """Typed configurations and the architecture registry."""
 from .guravik import GuravikConfig  # noqa: F401
+from .lotilix import LotilixConfig  # noqa: F401
 from .minimax_m3 import ConfigError, MiniMaxM3Config  # noqa: F401
 from .puvolix import PuvolixConfig  # noqa: F401
 from .tarulix import TarulixConfig  # noqa: F401

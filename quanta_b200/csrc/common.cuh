@@ -96,6 +96,11 @@ __device__ __forceinline__ float qb_warp_max(float v) {
   return v;
 }
 
+// the tanh form of gelu: z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float qb_gelu_tanh(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
 // Block-wide sum with a fixed order (thread partials -> warp tree -> warps in index order), so the
 // result for a row never depends on what else is in the batch.  `scratch` holds >= 32 floats.
 __device__ __forceinline__ float qb_block_sum(float v, float* scratch) {

@@ -4,9 +4,11 @@
 //
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (in this order)
 //
+// With a decay per key channel, g is a vector [D] per (token, head) and row i of S is multiplied by g[i].
+//
 // A first kernel turns the step's projections into what the chain reads: q and k of every (token, group) divided
 // by sqrt(sum of squares + unit_eps), q also times q_scale; beta = sigmoid(b); g = exp(-exp(A_log) * softplus(a +
-// dt_bias)); all float32.  The recurrence is a chain in time.  A column j of S never meets another column, so
+// dt_bias)), one number a head or D of them; all float32.  The recurrence is a chain in time.  A column j of S never meets another column, so
 // eight neighbouring lanes own one column (lane p the rows 4 (p + 8 j) .. + 3) in registers for the whole step, and a
 // block owns some columns of one (request, head).  Tokens are taken in chunks whose k, q, v, g and beta come into
 // shared memory by asynchronous copies while the chunk before is walked.  One token or a portion of a prompt is
@@ -16,16 +18,25 @@
 
 constexpr int GD_MAX_THREADS = 512;
 
-// One block a token.  qk: float32 rows [q (G x D) | k (G x D) | ...] (row stride qk_stride); ab: float32 rows whose
-// columns a_off + h and b_off + h hold the pre-activations of the decay and of beta (row stride ab_stride).
-__global__ void gated_delta_prep_kernel(const float* __restrict__ qk, int qk_stride, const float* __restrict__ ab,
-                                        int ab_stride, int a_off, int b_off, const float* __restrict__ A_log,
-                                        const float* __restrict__ dt_bias, float* __restrict__ q_out,
-                                        float* __restrict__ k_out, float* __restrict__ g_out,
-                                        float* __restrict__ beta_out, int T, int H, int G, int D, float q_scale,
-                                        float unit_eps) {
+// Block (t, y) of a token.  qk: float32 rows [q (G x D) | k (G x D) | ...] (row stride qk_stride); ab: float32 rows whose
+// column b_off + h holds the pre-activation of beta (row stride ab_stride); a: float32 rows (row stride a_stride) of the
+// decay's pre-activations, `per_head` numbers a head (1, or D for a decay per key channel), dt_bias laid out alike,
+// A_log one number a head.  The blocks of a token share its decays; the first one also does the unit vectors and beta.
+__global__ void gated_delta_prep_kernel(const float* __restrict__ qk, int qk_stride, const float* __restrict__ a,
+                                        int a_stride, const float* __restrict__ ab, int ab_stride, int b_off,
+                                        const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                                        float* __restrict__ q_out, float* __restrict__ k_out, float* __restrict__ g_out,
+                                        float* __restrict__ beta_out, int T, int H, int G, int D, int per_head,
+                                        float q_scale, float unit_eps) {
   const int t = blockIdx.x;
   if (t >= T) return;
+  const int n_g = H * per_head;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n_g; i += blockDim.x * gridDim.y) {
+    const float z = a[(size_t)t * a_stride + i] + dt_bias[i];
+    const float sp = z > 20.f ? z : log1pf(expf(z));
+    g_out[(size_t)t * n_g + i] = expf(-expf(A_log[i / per_head]) * sp);
+  }
+  if (blockIdx.y != 0) return;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   const float* row = qk + (size_t)t * qk_stride;
   for (int v = warp; v < 2 * G; v += nwarps) {          // v < G: the queries of group v; else the keys of group v - G
@@ -37,12 +48,8 @@ __global__ void gated_delta_prep_kernel(const float* __restrict__ qk, int qk_str
     float* dst = (v < G ? q_out + ((size_t)t * G + v) * D : k_out + ((size_t)t * G + (v - G)) * D);
     for (int i = lane; i < D; i += 32) dst[i] = src[i] * inv;
   }
-  for (int h = threadIdx.x; h < H; h += blockDim.x) {
-    const float a = ab[(size_t)t * ab_stride + a_off + h] + dt_bias[h];
-    const float sp = a > 20.f ? a : log1pf(expf(a));
-    g_out[(size_t)t * H + h] = expf(-expf(A_log[h]) * sp);
+  for (int h = threadIdx.x; h < H; h += blockDim.x)
     beta_out[(size_t)t * H + h] = 1.f / (1.f + expf(-ab[(size_t)t * ab_stride + b_off + h]));
-  }
 }
 
 __device__ __forceinline__ void gd_copy4(float* dst_smem, const float* src) {
@@ -55,8 +62,8 @@ __device__ __forceinline__ void gd_copy16(float* dst_smem, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 
-// GD_LANES neighbouring lanes own a column; RPT rows of it a lane: D <= GD_LANES * RPT
-template <int RPT, int GD_LANES>
+// GD_LANES neighbouring lanes own a column; RPT rows of it a lane: D <= GD_LANES * RPT; CH: a decay per key channel
+template <int RPT, int GD_LANES, bool CH>
 __global__ void __launch_bounds__(GD_MAX_THREADS, 1)
 gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_in, const float* __restrict__ v_in,
                    int v_stride, const float* __restrict__ g_in, const float* __restrict__ beta_in,
@@ -72,9 +79,10 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
   const int jl = tid / GD_LANES;
   const int j = col0 + jl;
   const bool owns = jl < cols_per_block && j < DV;
-  // a buffer: k [chunk, DP], q [chunk, DP], v [chunk, cols], g [chunk], beta [chunk]
+  // a buffer: k [chunk, DP], q [chunk, DP], with CH g [chunk, DP], v [chunk, cols], g [chunk], beta [chunk]
+  constexpr int PLANES = CH ? 3 : 2;
   const size_t plane = (size_t)chunk * DP;
-  const size_t buf_floats = 2 * plane + (size_t)chunk * cols_per_block + 2 * chunk;
+  const size_t buf_floats = PLANES * plane + (size_t)chunk * cols_per_block + 2 * chunk;
   // the padding rows (i >= D) are read as zeros and never written
   for (size_t i = tid; i < 2 * buf_floats; i += blockDim.x) sm[i] = 0.f;
 
@@ -90,7 +98,7 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
   }
   __syncthreads();
 
-  const bool wide = D % 4 == 0 && (((uintptr_t)k_in | (uintptr_t)q_in) & 15) == 0;
+  const bool wide = D % 4 == 0 && (((uintptr_t)k_in | (uintptr_t)q_in | (CH ? (uintptr_t)g_in : 0)) & 15) == 0;
   auto fetch = [&](int c0, int buf) {
     const int n = min(chunk, t1 - c0);
     float* b = sm + (size_t)buf * buf_floats;
@@ -102,6 +110,7 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
           const size_t gsrc = ((size_t)(c0 + tt) * G + grp) * D + i;
           gd_copy16(b + (size_t)tt * DP + i, k_in + gsrc);
           gd_copy16(b + plane + (size_t)tt * DP + i, q_in + gsrc);
+          if (CH) gd_copy16(b + 2 * plane + (size_t)tt * DP + i, g_in + ((size_t)(c0 + tt) * H + h) * D + i);
         }
       }
     } else {
@@ -111,17 +120,18 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
           const size_t gsrc = ((size_t)(c0 + tt) * G + grp) * D + i;
           gd_copy4(b + idx, k_in + gsrc);
           gd_copy4(b + plane + idx, q_in + gsrc);
+          if (CH) gd_copy4(b + 2 * plane + idx, g_in + ((size_t)(c0 + tt) * H + h) * D + i);
         }
       }
     }
-    float* bv = b + 2 * plane;
+    float* bv = b + PLANES * plane;
     for (int idx = tid; idx < n * cols_per_block; idx += blockDim.x) {
       const int tt = idx / cols_per_block, c = idx % cols_per_block;
       if (col0 + c < DV) gd_copy4(bv + idx, v_in + (size_t)(c0 + tt) * v_stride + (size_t)h * DV + col0 + c);
     }
     float* bg = bv + (size_t)chunk * cols_per_block;
     for (int tt = tid; tt < n; tt += blockDim.x) {
-      gd_copy4(bg + tt, g_in + (size_t)(c0 + tt) * H + h);
+      if (!CH) gd_copy4(bg + tt, g_in + (size_t)(c0 + tt) * H + h);
       gd_copy4(bg + chunk + tt, beta_in + (size_t)(c0 + tt) * H + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -135,19 +145,25 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
     if (c0 + chunk < t1) fetch(c0 + chunk, buf ^ 1);
     const float* s_k = sm + (size_t)buf * buf_floats;
     const float* s_q = s_k + plane;
-    const float* s_v = s_q + plane;
+    const float* s_gc = s_q + plane;                       // CH: the decays per channel
+    const float* s_v = s_k + PLANES * plane;
     const float* s_g = s_v + (size_t)chunk * cols_per_block;
     const float* s_b = s_g + chunk;
     for (int tt = 0; tt < n; ++tt) {
       const size_t o = (size_t)tt * DP;
-      const float g = s_g[tt], beta = s_b[tt];
+      const float g = CH ? 1.f : s_g[tt], beta = s_b[tt];
       // four partial sums a dot product: the chain of dependent additions is a quarter as long
       float d4[4] = {0.f, 0.f, 0.f, 0.f};
       float4 k4[RPT / 4];
 #pragma unroll
       for (int jj = 0; jj < RPT / 4; ++jj) {
         k4[jj] = *reinterpret_cast<const float4*>(s_k + o + 4 * (p + GD_LANES * jj));
-        col[4 * jj + 0] *= g; col[4 * jj + 1] *= g; col[4 * jj + 2] *= g; col[4 * jj + 3] *= g;
+        if (CH) {
+          const float4 g4 = *reinterpret_cast<const float4*>(s_gc + o + 4 * (p + GD_LANES * jj));
+          col[4 * jj + 0] *= g4.x; col[4 * jj + 1] *= g4.y; col[4 * jj + 2] *= g4.z; col[4 * jj + 3] *= g4.w;
+        } else {
+          col[4 * jj + 0] *= g; col[4 * jj + 1] *= g; col[4 * jj + 2] *= g; col[4 * jj + 3] *= g;
+        }
         d4[0] += k4[jj].x * col[4 * jj + 0];
         d4[1] += k4[jj].y * col[4 * jj + 1];
         d4[2] += k4[jj].z * col[4 * jj + 2];
@@ -187,18 +203,20 @@ gated_delta_kernel(const float* __restrict__ q_in, const float* __restrict__ k_i
 }
 
 // qkv: float32 rows [q (G x D) | k (G x D) | v (H x DV)] after convolution and activation (row stride qkv_stride);
-// ab: float32 rows with the pre-activations of decay (a_off + h) and beta (b_off + h); scratch: T * (2 G D + 2 H)
-// floats; out: float32 [T, H, DV].
-extern "C" int qb_gated_delta(const float* qkv, int qkv_stride, const float* ab, int ab_stride, int a_off, int b_off,
-                              const float* A_log, const float* dt_bias, float* state, float* out, float* scratch,
-                              const int* req_start, const int* req_slot, int R, int T, int H, int G, int D, int DV,
-                              float q_scale, float unit_eps, cudaStream_t stream) {
+// a: float32 rows of the decay's pre-activations, one a head or (per_channel) D a head; ab: float32 rows with the
+// pre-activations of beta (b_off + h); scratch: T * (2 G D + H (per_channel ? D : 1) + H) floats; out: float32 [T, H, DV].
+extern "C" int qb_gated_delta(const float* qkv, int qkv_stride, const float* a, int a_stride, const float* ab,
+                              int ab_stride, int b_off, int per_channel, const float* A_log, const float* dt_bias,
+                              float* state, float* out, float* scratch, const int* req_start, const int* req_slot, int R,
+                              int T, int H, int G, int D, int DV, float q_scale, float unit_eps, cudaStream_t stream) {
   if (R <= 0 || T <= 0) return 0;
   if (D <= 0 || D > 256 || DV <= 0 || DV > 256 || H <= 0 || G <= 0 || H % G) return QB_ERR_UNSUPPORTED;
   const size_t n = (size_t)T * G * D;
-  float *q_s = scratch, *k_s = scratch + n, *g_s = scratch + 2 * n, *b_s = g_s + (size_t)T * H;
-  gated_delta_prep_kernel<<<T, 128, 0, stream>>>(qkv, qkv_stride, ab, ab_stride, a_off, b_off, A_log, dt_bias, q_s, k_s,
-                                                 g_s, b_s, T, H, G, D, q_scale, unit_eps);
+  const int per_head = per_channel ? D : 1;
+  float *q_s = scratch, *k_s = scratch + n, *g_s = scratch + 2 * n, *b_s = g_s + (size_t)T * H * per_head;
+  const dim3 pgrid(T, T >= 512 ? 1 : min(32, (H * per_head + 255) / 256));
+  gated_delta_prep_kernel<<<pgrid, 256, 0, stream>>>(qkv, qkv_stride, a, a_stride, ab, ab_stride, b_off, A_log, dt_bias,
+                                                     q_s, k_s, g_s, b_s, T, H, G, D, per_head, q_scale, unit_eps);
   QB_LAUNCH_CHECK();
   // eight lanes a column.  Sixteen (half the multiply-adds a lane and token for one more step of the sums) were
   // measured: no faster on a prompt (637 against 631 us for 2,048 tokens, 16 heads of 128 x 128) and slower for single
@@ -218,12 +236,12 @@ extern "C" int qb_gated_delta(const float* qkv, int qkv_stride, const float* ab,
   const int rpt = per_lane <= 4 ? 4 : per_lane <= 8 ? 8 : per_lane <= 16 ? 16 : 32;
   const int dp = rpt * lanes;
   const int chunk = dp <= 128 ? 16 : 8;
-  const size_t smem = (size_t)2 * (2 * chunk * dp + chunk * cols + 2 * chunk) * sizeof(float);
+  const size_t smem = (size_t)2 * ((per_channel ? 3 : 2) * chunk * dp + chunk * cols + 2 * chunk) * sizeof(float);
   dim3 grid(R, H, splits);
   const float* v_in = qkv + (size_t)2 * G * D;
-#define GD_LAUNCH(N, L)                                                                                    \
+#define GD_LAUNCH_AS(N, L, CH)                                                                              \
   do {                                                                                                     \
-    auto kern = gated_delta_kernel<N, L>;                                                                  \
+    auto kern = gated_delta_kernel<N, L, CH>;                                                                \
     if (smem > 48 * 1024) {                                                                                \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
       if (e != cudaSuccess) return (int)e;                                                                 \
@@ -231,11 +249,17 @@ extern "C" int qb_gated_delta(const float* qkv, int qkv_stride, const float* ab,
     kern<<<grid, threads, smem, stream>>>(q_s, k_s, v_in, qkv_stride, g_s, b_s, state, out, req_start,     \
                                           req_slot, H, G, D, DV, cols, chunk);                             \
   } while (0)
+#define GD_LAUNCH(N, L)                   \
+  do {                                    \
+    if (per_channel) GD_LAUNCH_AS(N, L, true); \
+    else GD_LAUNCH_AS(N, L, false);       \
+  } while (0)
   if (rpt == 4) GD_LAUNCH(4, 8);
   else if (rpt == 8) GD_LAUNCH(8, 8);
   else if (rpt == 16) GD_LAUNCH(16, 8);
   else GD_LAUNCH(32, 8);
 #undef GD_LAUNCH
+#undef GD_LAUNCH_AS
   QB_LAUNCH_CHECK();
   return 0;
 }

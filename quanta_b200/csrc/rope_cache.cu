@@ -5,14 +5,16 @@
 // step; a layer that reads another layer's cache has rows [q | anything else] (has_kv = 0).  For each token:
 //   q, k  <- RMSNorm (none | over all heads of the row | per head), float32
 //            (src/quanta/minimax/model_m3.py:15-17 / src/quanta/minimax/attention.py:172-182)
-//   q, k  <- rotate-half on the first `rd` dims of each head, pair j using position axis
-//            pair_axis[j] and angle float(pos) * inv_freq[j]  (src/quanta/minimax/model_m3.py:83-96)
+//   q, k  <- rotation of the first `rd` dims of each head, pair j using position axis pair_axis[j] and angle
+//            float(pos) * inv_freq[j]; pair j is the dims (j, j + rd/2)  (src/quanta/minimax/model_m3.py:83-96), or
+//            with `interleaved` the neighbours (2j, 2j + 1)
 //   q     <- q * (1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1))     (temp_every > 0: a query
 //            temperature that grows with the position, float32)
 //   q     <- q * head_scale[head]          (head_scale: a float32 number per q head that multiplies the head's
 //            scores; null for none)
 //   v     <- (1 - lambda) v + lambda v_first      (v_first: float32 values [T, nkv * vd] that an earlier layer left for
 //            the same tokens, lambda one number on the device; v_export: this layer leaves its own values there)
+//   v     =  the projected k before norm and rotation (tied_v: the rows are [q | k | anything else], vd == hd)
 //   q     -> q_out [T, nq, hd];  k -> pages [page, kv_head, slot, hd], v -> pages [page, kv_head, slot, vd]
 //            through the block table (keys and values may have different head sizes)
 // The rows may be float32 accumulators of the projection while q and the cache are in the activation dtype, and a
@@ -31,7 +33,7 @@ __global__ void qknorm_rope_write_kernel(
     const float* __restrict__ inv_freq, const int* __restrict__ pair_axis,
     const int* __restrict__ positions, int n_axes, const int* __restrict__ tok_pos,
     const int* __restrict__ tok_req, const int* __restrict__ block_table, int bt_stride, int T, int nq,
-    int nkv_all, int hd, int vd, int has_kv, int rd, float temp_coef, int temp_every, int page_size, int num_pages,
+    int nkv_all, int hd, int vd, int has_kv, int tied_v, int rd, int interleaved, float temp_coef, int temp_every, int page_size, int num_pages,
     int vec, const float* __restrict__ bias, const float* __restrict__ v_first, const float* __restrict__ v_lambda,
     float* __restrict__ v_export, const float* __restrict__ head_scale, int* status) {
   extern __shared__ float smem[];
@@ -142,10 +144,11 @@ __global__ void qknorm_rope_write_kernel(
   // rotation: each (head, pair) is owned by one thread
   for (int i = threadIdx.x; i < (nq + nkv) * half; i += blockDim.x) {
     const int h = i / half, j = i % half;
-    const float a = buf[h * hd + j], b = buf[h * hd + half + j];
+    const int ia = h * hd + (interleaved ? 2 * j : j), ib = interleaved ? ia + 1 : ia + half;
+    const float a = buf[ia], b = buf[ib];
     const float c = cs[j], s = cs[half + j];
-    buf[h * hd + j] = a * c - b * s;
-    buf[h * hd + half + j] = b * c + a * s;
+    buf[ia] = a * c - b * s;
+    buf[ib] = b * c + a * s;
   }
   if (half > 0) __syncthreads();
 
@@ -171,8 +174,8 @@ __global__ void qknorm_rope_write_kernel(
     return;
   }
   const int slot = pos % page_size;
-  const IN* vrow = row + qn + kn;
-  const float* vbias = bias != nullptr ? bias + qn + kn : nullptr;
+  const IN* vrow = row + qn + (tied_v ? 0 : kn);
+  const float* vbias = bias != nullptr ? bias + qn + (tied_v ? 0 : kn) : nullptr;
   const float lam = v_first != nullptr ? v_lambda[0] : 0.f;
   const float* vf = v_first != nullptr ? v_first + (size_t)t * vn : nullptr;
   float* vx = v_export != nullptr ? v_export + (size_t)t * vn : nullptr;
@@ -218,8 +221,8 @@ extern "C" int qb_qknorm_rope_write(
     const void* qkv, int in_dtype, int dtype, int row_stride, void* q_out, void* k_cache, void* v_cache, const float* q_norm_w,
     const float* k_norm_w, int norm_kind, float eps, const float* inv_freq, const int* pair_axis,
     const int* positions, int n_axes, const int* tok_pos, const int* tok_req, const int* block_table,
-    int bt_stride, int T, int nq, int nkv, int hd, int vd, int has_kv, int rd, float temp_coef, int temp_every,
-    int page_size, int num_pages, const float* bias, const float* v_first, const float* v_lambda, float* v_export,
+    int bt_stride, int T, int nq, int nkv, int hd, int vd, int has_kv, int tied_v, int rd, int interleaved, float temp_coef,
+    int temp_every, int page_size, int num_pages, const float* bias, const float* v_first, const float* v_lambda, float* v_export,
     const float* head_scale, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rd % 2 || rd > hd || rd < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || hd <= 0 || vd <= 0) return QB_ERR_BAD_ARG;
@@ -231,7 +234,8 @@ extern "C" int qb_qknorm_rope_write(
   if (in_dtype != dtype && in_dtype != QB_F32) return QB_ERR_BAD_ARG;
   if (!has_kv && k_cache != nullptr) return QB_ERR_BAD_ARG;
   const int nk = has_kv ? nkv : 0;
-  if (row_stride < nq * hd + nk * (hd + vd)) return QB_ERR_BAD_ARG;
+  if (tied_v && (vd != hd || !has_kv)) return QB_ERR_BAD_ARG;
+  if (row_stride < nq * hd + nk * (hd + (tied_v ? 0 : vd))) return QB_ERR_BAD_ARG;
   // rows are moved in 16-byte pieces where every piece starts on such a boundary; else element by element
   const int vec = (hd % 8 == 0 && vd % 8 == 0 && row_stride % 8 == 0 && ((uintptr_t)qkv & 15) == 0) ? 1 : 0;
   const size_t smem = (size_t)((nq + nk) * hd + rd + 32 + nq + nk) * sizeof(float);
@@ -245,8 +249,8 @@ extern "C" int qb_qknorm_rope_write(
     }                                                                                                           \
     kern<<<T, threads, smem, stream>>>((const IN*)qkv, row_stride, (A*)q_out, (A*)k_cache, (A*)v_cache, q_norm_w, \
                                        k_norm_w, norm_kind, eps, inv_freq, pair_axis, positions, n_axes, tok_pos, \
-                                       tok_req, block_table, bt_stride, T, nq, nkv, hd, vd, has_kv, rd, temp_coef, \
-                                       temp_every, page_size, num_pages, vec, bias, v_first, v_lambda, v_export,  \
+                                       tok_req, block_table, bt_stride, T, nq, nkv, hd, vd, has_kv, tied_v, rd,  \
+                                       interleaved, temp_coef, temp_every, page_size, num_pages, vec, bias, v_first, v_lambda, v_export,  \
                                        head_scale, status);                                                              \
   } while (0)
   // steps of few tokens: more threads a token, so that each of the kernel's phases is short

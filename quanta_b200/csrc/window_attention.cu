@@ -1,7 +1,8 @@
 // Sliding-window attention over the paged cache with optional extras, SIMT version (float32 arithmetic
 // throughout; the cache, q and out are float32 or bfloat16).
 //
-// Token t of request r at position p reads the keys [p - window + 1, p] of r's pages (window 0: [0, p]) and,
+// Token t of request r at position p reads the keys [p - window + 1, p] of r's pages (window 0: [0, p]), or with
+// `chunk` only those of p's own chunk, [floor(p / chunk) * chunk, p] (chunks are counted from position 0), and,
 // when the layer keeps pooled blocks, one key and one value per block of `pool` tokens that lies wholly before
 // the window (block b holds positions b*pool .. b*pool + pool - 1 and is read when b*pool + pool - 1 <= p -
 // window).  Tokens and blocks share one softmax.  Per (query head h, key j):
@@ -54,7 +55,7 @@ struct WaParams {
   int pool_stride;
   int T, nq, nkv, hd, vd, page_size, num_pages, num_pool_pages;
   float scale, cap;
-  int window, pool;
+  int window, pool, chunk;     // chunk > 0: a token sees its own chunk of that many positions only
   const float* dist_bias;      // [window, nq] or null
   const float* sink;           // [nq] or null
   int all_values;              // 1: every head's weights on the values of all kv heads (scratch), 0: its own
@@ -63,6 +64,13 @@ struct WaParams {
   float* part;                 // sum, sums of values) in `part` [T, nq, n_split, 2 + (all_values ? nkv : 1) * vd]
   int* status;
 };
+
+// the first position that a token at `pos` sees
+__device__ __forceinline__ int wa_first_seen(const WaParams& P, int pos) {
+  int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+  if (P.chunk > 0) lo = max(lo, pos / P.chunk * P.chunk);
+  return lo;
+}
 
 // NV: value chunks of 32 a lane holds, ceil(vd / 32)
 template <typename A, int NV>
@@ -90,7 +98,7 @@ window_attention_kernel(const A* __restrict__ q, const A* __restrict__ k_cache, 
   const int req = P.tok_req[t];
   const int* bt = P.block_table + (size_t)req * P.bt_stride;
   const int* pt = P.pool_table ? P.pool_table + (size_t)req * P.pool_stride : nullptr;
-  const int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+  const int lo = wa_first_seen(P, pos);
   // pooled blocks that lie wholly before the window: b * pool + pool - 1 <= pos - window
   const int n_blocks = (pt != nullptr && P.window > 0 && pos - P.window + 1 >= P.pool) ? (pos - P.window + 1) / P.pool : 0;
   const int n_keys = n_blocks + (pos - lo + 1);
@@ -228,7 +236,7 @@ window_attention_ranges_kernel(const A* __restrict__ q, const A* __restrict__ k_
   const int req = P.tok_req[t];
   const int* bt = P.block_table + (size_t)req * P.bt_stride;
   const int* pt = P.pool_table ? P.pool_table + (size_t)req * P.pool_stride : nullptr;
-  const int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+  const int lo = wa_first_seen(P, pos);
   const int n_blocks = (pt != nullptr && P.window > 0 && pos - P.window + 1 >= P.pool) ? (pos - P.window + 1) / P.pool : 0;
   const int n_keys = n_blocks + (pos - lo + 1);
   const int per_split = ((n_keys + P.n_split - 1) / P.n_split + 31) / 32 * 32;
@@ -415,19 +423,19 @@ extern "C" int qb_window_attention(const void* q, int dtype, const void* k_cache
                                    const float* talk, const int* tok_pos, const int* tok_req, const int* block_table,
                                    int bt_stride, const int* pool_table, int pool_stride, int T, int nq, int nkv,
                                    int hd, int vd, int page_size, int num_pages, int num_pool_pages, float scale,
-                                   float cap, int window, int pool, const float* dist_bias, const float* sink,
+                                   float cap, int window, int pool, int chunk, const float* dist_bias, const float* sink,
                                    float* part, int n_split, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (n_split < 1 || (n_split > 1 && part == nullptr)) return QB_ERR_BAD_ARG;
   if (hd <= 0 || vd <= 0 || hd > WA_MAX_HD || vd > WA_MAX_HD || nq % nkv || page_size <= 0) return QB_ERR_UNSUPPORTED;
   if (pool_table != nullptr && (pool <= 0 || window <= 0 || kp_cache == nullptr || vp_cache == nullptr)) return QB_ERR_BAD_ARG;
-  if (dist_bias != nullptr && window <= 0) return QB_ERR_BAD_ARG;
+  if ((dist_bias != nullptr && window <= 0) || chunk < 0 || (chunk > 0 && pool_table != nullptr)) return QB_ERR_BAD_ARG;
   if (talk != nullptr && scratch == nullptr) return QB_ERR_BAD_ARG;
   WaParams P;
   P.tok_pos = tok_pos; P.tok_req = tok_req; P.block_table = block_table; P.bt_stride = bt_stride;
   P.pool_table = pool_table; P.pool_stride = pool_stride;
   P.T = T; P.nq = nq; P.nkv = nkv; P.hd = hd; P.vd = vd; P.page_size = page_size; P.num_pages = num_pages;
-  P.num_pool_pages = num_pool_pages; P.scale = scale; P.cap = cap; P.window = window; P.pool = pool;
+  P.num_pool_pages = num_pool_pages; P.scale = scale; P.cap = cap; P.window = window; P.pool = pool; P.chunk = chunk;
   P.dist_bias = dist_bias; P.sink = sink; P.all_values = talk != nullptr; P.status = status;
   P.vec = (hd % 8 == 0 && ((uintptr_t)k_cache & 15) == 0 && (kp_cache == nullptr || ((uintptr_t)kp_cache & 15) == 0)) ? 1 : 0;
   P.n_split = n_split; P.part = part;
@@ -645,8 +653,8 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int r_a = warp * 16 + g8, r_b = r_a + 8;
   const int pos_a = s_pos[r_a], pos_b = s_pos[r_b];
   const int req_a = s_req[r_a], req_b = s_req[r_b];
-  const int lo_a = (P.window > 0 && pos_a - P.window + 1 > 0) ? pos_a - P.window + 1 : 0;
-  const int lo_b = (P.window > 0 && pos_b - P.window + 1 > 0) ? pos_b - P.window + 1 : 0;
+  const int lo_a = wa_first_seen(P, pos_a);
+  const int lo_b = wa_first_seen(P, pos_b);
   const bool pooling = P.pool_table != nullptr && P.window > 0;
   const int nb_a = (pooling && pos_a - P.window + 1 >= P.pool) ? (pos_a - P.window + 1) / P.pool : 0;
   const int nb_b = (pooling && pos_b - P.window + 1 >= P.pool) ? (pos_b - P.window + 1) / P.pool : 0;
@@ -665,7 +673,7 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     int lo_min = 0x7fffffff, pos_max = -1, nb_max = 0;
     for (int r = ra; r < rb; ++r) {
       const int p = s_pos[r];
-      const int lo = (P.window > 0 && p - P.window + 1 > 0) ? p - P.window + 1 : 0;
+      const int lo = wa_first_seen(P, p);
       const int nb = (pooling && p - P.window + 1 >= P.pool) ? (p - P.window + 1) / P.pool : 0;
       lo_min = min(lo_min, lo); pos_max = max(pos_max, p); nb_max = max(nb_max, nb);
     }
@@ -892,20 +900,20 @@ extern "C" int qb_window_attention_mma(const void* q, int dtype, const void* k_c
                                        const float* talk, const int* tok_pos, const int* tok_req, const int* block_table,
                                        int bt_stride, const int* pool_table, int pool_stride, int T, int nq, int nkv,
                                        int hd, int vd, int page_size, int num_pages, int num_pool_pages, float scale,
-                                       float cap, int window, int pool, const float* dist_bias, const float* sink,
+                                       float cap, int window, int pool, int chunk, const float* dist_bias, const float* sink,
                                        int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (!qb_window_attention_mma_supported(dtype, hd, vd) || nq % nkv || page_size <= 0 || nq > 65535 || nkv > 65535)
     return QB_ERR_UNSUPPORTED;
   if (pool_table != nullptr && (pool <= 0 || window <= 0 || kp_cache == nullptr || vp_cache == nullptr)) return QB_ERR_BAD_ARG;
-  if (dist_bias != nullptr && window <= 0) return QB_ERR_BAD_ARG;
+  if ((dist_bias != nullptr && window <= 0) || chunk < 0 || (chunk > 0 && pool_table != nullptr)) return QB_ERR_BAD_ARG;
   if (talk != nullptr && scratch == nullptr) return QB_ERR_BAD_ARG;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)kp_cache | (uintptr_t)vp_cache) & 15) return QB_ERR_BAD_ARG;
   WaParams P;
   P.tok_pos = tok_pos; P.tok_req = tok_req; P.block_table = block_table; P.bt_stride = bt_stride;
   P.pool_table = pool_table; P.pool_stride = pool_stride;
   P.T = T; P.nq = nq; P.nkv = nkv; P.hd = hd; P.vd = vd; P.page_size = page_size; P.num_pages = num_pages;
-  P.num_pool_pages = num_pool_pages; P.scale = scale; P.cap = cap; P.window = window; P.pool = pool;
+  P.num_pool_pages = num_pool_pages; P.scale = scale; P.cap = cap; P.window = window; P.pool = pool; P.chunk = chunk;
   P.dist_bias = dist_bias; P.sink = sink; P.all_values = talk != nullptr; P.status = status; P.vec = 1;
   P.n_split = 1; P.part = nullptr;
   const size_t smem = ((size_t)(WM_BM + 2 * WM_BN) * (hd + 8) + (size_t)2 * WM_BN * (vd + 8)) * 2 + 2 * WM_BN * sizeof(long long)

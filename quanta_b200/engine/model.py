@@ -15,7 +15,7 @@ import torch
 from .. import kernels, matmul
 from ..config.registry import load_config
 from ..parts import block as _block  # noqa: F401  (registers the built-in block, embedding and head)
-from ..parts.base import CacheSpec, Part, StreamCopy, StreamsPending, TensorSpec, make
+from ..parts.base import Addends, CacheSpec, Part, StreamCopy, StreamsPending, TensorSpec, make
 from ..parts.spec import ModelSpec
 from ..weights.loader import FolderSource, RandomSource, open_fetch
 from ..weights.safetensors_io import write_safetensors
@@ -36,6 +36,8 @@ def _plain(pending):
     stream is no contribution)."""
     if isinstance(pending, StreamCopy):
         return None
+    if isinstance(pending, Addends):
+        return pending.total()
     return pending.materialize() if hasattr(pending, "materialize") else pending
 
 
@@ -127,6 +129,7 @@ class Model:
     def forward(self, token_ids, ctx, caches, states, want_rows):
         """``token_ids`` int32 [T]; ``caches[pos]``/``states[pos]`` per schedule position; ``want_rows``
         int32 rows whose logits are returned ([n, vocab] float32) or None."""
+        ctx.token_ids = token_ids
         h = self.embedding.forward(token_ids, ctx)
         embedded = h.clone() if any(e.add_embedding for e in self.schedule) else None
         pending = None

@@ -273,7 +273,7 @@ def qknorm_rope_write(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, norm_kin
                       inv_freq, pair_axis, positions, tok_pos, tok_req, block_table, nq: int, nkv: int,
                       hd: int, rd: int, page_size: int, status, *, vd: int | None = None, has_kv: bool = True,
                       q_temp_coef: float = 0.0, q_temp_every: int = 0, bias=None, v_first=None, v_lambda=None,
-                      v_export=None, head_scale=None) -> None:
+                      v_export=None, head_scale=None, interleaved: bool = False, tied_values: bool = False) -> None:
     """Rows ``[q | k | v | ...]`` of a fused projection (``qkv`` may be wider than the three; its row stride is
     honoured) -> normed, rotated queries in ``q_out`` and keys / values in the pages.  ``vd``: the values' head
     size when it differs from ``hd``; ``has_kv`` False: the rows start with q alone (a layer that reads another
@@ -283,10 +283,15 @@ def qknorm_rope_write(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, norm_kin
     (both None).  ``v_first`` (float32 ``[T, nkv * vd]``) with ``v_lambda`` (one float32 on the device): the values
     become ``(1 - lambda) v + lambda v_first`` before they are cached; ``v_export``: this layer's own values (bias
     added, not blended) are left there as float32.  ``head_scale`` (float32 ``[nq]``): a number per q head that
-    multiplies the head's queries (and so its scores) after norm and rotation."""
+    multiplies the head's queries (and so its scores) after norm and rotation.  ``interleaved``: the rotated pairs are
+    the neighbours ``(2j, 2j + 1)`` instead of ``(j, j + rd/2)``.  ``tied_values``: the rows are ``[q | k | ...]`` and the
+    values are the projected keys before norm and rotation (``vd`` equals ``hd``)."""
     T = qkv.shape[0]
     vd = hd if vd is None else int(vd)
-    if qkv.stride(1) != 1 or qkv.shape[1] < nq * hd + (nkv * (hd + vd) if has_kv else 0):
+    if tied_values and (vd != hd or not has_kv):
+        raise ValueError("qknorm_rope_write: values that are the keys have the keys' size and belong to the layer")
+    n_row = nq * hd + (nkv * (hd + (0 if tied_values else vd)) if has_kv else 0)
+    if qkv.stride(1) != 1 or qkv.shape[1] < n_row:
         raise ValueError("qknorm_rope_write: qkv width mismatch")
     if (q_out.dtype != qkv.dtype and qkv.dtype != torch.float32) or q_out.numel() != T * nq * hd:
         raise ValueError("qknorm_rope_write: q_out mismatch")
@@ -300,7 +305,6 @@ def qknorm_rope_write(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, norm_kin
                 or k_cache.shape[0] != v_cache.shape[0]):
             raise ValueError("qknorm_rope_write: cache shape mismatch")
         num_pages = k_cache.shape[0]
-    n_row = nq * hd + (nkv * (hd + vd) if has_kv else 0)
     for t, n, size in ((bias, "bias", n_row), (v_first, "v_first", T * nkv * vd), (v_lambda, "v_lambda", 1),
                        (v_export, "v_export", T * nkv * vd), (head_scale, "head_scale", nq)):
         if t is not None:
@@ -325,7 +329,8 @@ def qknorm_rope_write(qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, norm_kin
         ctypes.c_void_p(qkv.data_ptr()), _code(qkv), _code(q_out), int(qkv.stride(0)), _p(q_out), _p(k_cache), _p(v_cache),
         _p(q_norm_w), _p(k_norm_w) if has_kv else ctypes.c_void_p(0), norm_kind,
         ctypes.c_float(eps), _p(inv_freq), _p(pair_axis), _p(positions), n_axes, _p(tok_pos), _p(tok_req),
-        _p(block_table), block_table.shape[1], T, nq, nkv, hd, vd, int(has_kv), rd, ctypes.c_float(q_temp_coef),
+        _p(block_table), block_table.shape[1], T, nq, nkv, hd, vd, int(has_kv), int(tied_values), rd,
+        int(interleaved), ctypes.c_float(q_temp_coef),
         int(q_temp_every), page_size, num_pages, _p(bias), _p(v_first), _p(v_lambda), _p(v_export), _p(head_scale),
         _p(status), _stream()), "qknorm_rope_write")
 
@@ -778,34 +783,58 @@ def tanh_cols(x, off: int, n: int, out) -> None:
 LATENT_MAX_RANK = 512
 
 
+def _rows_of(t, width: int, name: str):
+    """(pointer, row stride) of float32 rows that may be a column range of wider rows."""
+    _want(t, torch.float32, name)
+    if t.dim() != 2 or t.shape[1] != width or t.stride(1) != 1 or not t.is_cuda:
+        raise ValueError(f"{name}: rows of {width} contiguous numbers on the device are wanted")
+    return ctypes.c_void_p(t.data_ptr()), int(t.stride(0))
+
+
 def latent_write(dkv, gain, inv_freq, cache, tok_pos, tok_req, block_table, rank: int, rot: int, rotated: int,
-                 page_size: int, eps: float, status) -> None:
+                 page_size: int, eps: float, status, *, interleaved: bool = False, q_down=None, q_gain=None,
+                 q_out=None) -> None:
     """Rows ``[T, rank + rot]`` float32 -> the cache rows of their positions: RMS norm with ``gain`` of the
-    first ``rank``, rotation by the position of the first ``rotated`` of the last ``rot``.  ``cache`` ``[pages, 1, page_size, rank + rot]``."""
-    _want(dkv, torch.float32, "dkv"); _want(gain, torch.float32, "gain"); _want(inv_freq, torch.float32, "inv_freq")
-    T = dkv.shape[0]
-    if (dkv.shape[1] != rank + rot or gain.numel() != rank or inv_freq.numel() != rotated // 2
-            or tuple(cache.shape[1:]) != (1, page_size, rank + rot)):
-        raise ValueError("latent_write: shape mismatch")
-    _check(lib().qb_latent_write(_p(dkv), _p(gain), _p(inv_freq), _p(cache), _code(cache), _p(tok_pos), _p(tok_req),
-                                 _p(block_table), block_table.shape[1], T, rank, rot, int(rotated), page_size,
-                                 cache.shape[0], ctypes.c_float(eps), _p(status), _stream()), "latent_write")
+    first ``rank``, rotation by the position of the first ``rotated`` of the last ``rot`` (pairs ``(i, i + rotated/2)``
+    or, ``interleaved``, neighbours).  ``cache`` ``[pages, 1, page_size, rank + rot]``.  In the same launch, with
+    ``q_down`` (float32 ``[T, q_rank]``): ``q_out = q_gain * q_down / rms(q_down)``.  Both kinds of rows may be column
+    ranges of wider rows; ``dkv`` None: only the second is done."""
+    T = (dkv if dkv is not None else q_down).shape[0]
+    dkv_p, dkv_s, dq_p, dq_s, q_rank = ctypes.c_void_p(0), 0, ctypes.c_void_p(0), 0, 0
+    if dkv is not None:
+        dkv_p, dkv_s = _rows_of(dkv, rank + rot, "dkv")
+        _want(gain, torch.float32, "gain"); _want(inv_freq, torch.float32, "inv_freq")
+        if (gain.numel() != rank or inv_freq.numel() != rotated // 2
+                or tuple(cache.shape[1:]) != (1, page_size, rank + rot)):
+            raise ValueError("latent_write: shape mismatch")
+    if q_down is not None:
+        q_rank = q_down.shape[1]
+        dq_p, dq_s = _rows_of(q_down, q_rank, "q_down")
+        _want(q_gain, torch.float32, "q_gain")
+        if q_gain.numel() != q_rank or tuple(q_out.shape) != (T, q_rank) or q_out.dtype != cache.dtype:
+            raise ValueError("latent_write: shape mismatch of the queries' latent")
+    _check(lib().qb_latent_write(dkv_p, dkv_s, _p(gain), _p(inv_freq), _p(cache), _code(cache), dq_p, dq_s, _p(q_gain),
+                                 _p(q_out), q_rank, _p(tok_pos), _p(tok_req), _p(block_table), block_table.shape[1], T,
+                                 rank, rot, int(rotated), int(interleaved), page_size, cache.shape[0],
+                                 ctypes.c_float(eps), _p(status), _stream()), "latent_write")
 
 
-def latent_query(q, inv_freq, q_plain, q_rot, tok_pos, n_heads: int, dim: int, rot: int, rotated: int) -> None:
+def latent_query(q, inv_freq, q_plain, q_rot, tok_pos, n_heads: int, dim: int, rot: int, rotated: int,
+                 interleaved: bool = False) -> None:
     """``q`` float32 ``[T, heads, dim + rot]`` -> ``q_plain`` ``[heads, T, dim]`` and ``q_rot`` float32
-    ``[T, heads, rot]``, its first ``rotated`` dimensions rotated by the position."""
+    ``[T, heads, rot]``, its first ``rotated`` dimensions rotated by the position (pairs as in ``latent_write``)."""
     _want(q, torch.float32, "q"); _want(q_rot, torch.float32, "q_rot")
     T = q.shape[0]
     if q.numel() != T * n_heads * (dim + rot) or q_plain.numel() != T * n_heads * dim or q_rot.numel() != T * n_heads * rot:
         raise ValueError("latent_query: shape mismatch")
     _check(lib().qb_latent_query(_p(q), _p(inv_freq), _p(q_plain), _code(q_plain), _p(q_rot), _p(tok_pos), T, n_heads,
-                                 dim, rot, int(rotated), _stream()), "latent_query")
+                                 dim, rot, int(rotated), int(interleaved), _stream()), "latent_query")
 
 
 def latent_attend_uses_tensor_cores(cache_dtype, rank: int, rot: int) -> bool:
-    """Whether ``latent_attend`` runs these shapes on the tensor cores (bfloat16 cache, rank 64/128/256/512, rot a
-    multiple of 16) or on the CUDA cores (float32 arithmetic; every other shape, and the float32 path)."""
+    """Whether ``latent_attend`` runs these shapes on the tensor cores (bfloat16 cache, rank a multiple of 8 up to
+    512, rank + rot a multiple of 16) or on the CUDA cores (float32 arithmetic; every other shape, and the float32
+    path)."""
     return cache_dtype == torch.bfloat16 and bool(lib().qb_latent_attend_mma_supported(int(rank), int(rot)))
 
 
@@ -813,13 +842,17 @@ LATENT_MMA_ROWS = 32        # (token, head) rows a block of the tensor-core kern
 
 
 def latent_attend(q_lat, q_rot, cache, sink, out, tok_pos, tok_req, block_table, scale: float, n_ranges: int,
-                  status, req_start=None, tensor_cores: bool | None = None) -> None:
+                  status, req_start=None, tensor_cores: bool | None = None, *, window: int = 0, gate=None,
+                  float32_weights: bool = False) -> None:
     """Causal softmax attention of every token and head over the cached latent rows, with an optional sink.
     ``q_lat`` ``[heads, T, rank]``, ``q_rot`` float32 ``[T, heads, rot]``, ``out`` ``[heads, T, rank]``; each
     token's keys are cut into ``n_ranges`` ranges that run as blocks of their own and are merged in order.
+    ``window`` > 0: a token sees the last ``window`` positions only.  ``gate`` (float32 ``[T, heads]``, possibly a
+    column range of wider rows): a head's result is multiplied by ``sigmoid(gate)``.
     With ``req_start`` (int32 ``[requests + 1]``, the step's token rows of each request; token ``t`` belongs to
     request ``tok_req[t]``) and shapes that ``latent_attend_uses_tensor_cores`` takes, the scores and sums run on
-    the tensor cores; ``tensor_cores`` False keeps them on the CUDA cores."""
+    the tensor cores; ``tensor_cores`` False keeps them on the CUDA cores.  ``float32_weights``: the tensor cores take
+    the softmax weights in two bfloat16 parts instead of one."""
     H, T, C = q_lat.shape
     num_pages, one, page_size, W = cache.shape
     R = W - C
@@ -827,25 +860,31 @@ def latent_attend(q_lat, q_rot, cache, sink, out, tok_pos, tok_req, block_table,
         raise ValueError("latent_attend: shape/dtype mismatch")
     if sink is not None:
         _want(sink, torch.float32, "sink")
-    part = torch.empty(T * H * n_ranges * (C + 2), dtype=torch.float32, device=q_lat.device)
+    gate_p, gate_s = (ctypes.c_void_p(0), 0) if gate is None else _rows_of(gate, H, "gate")
     mma = (req_start is not None and q_lat.dtype == torch.float32 and tensor_cores is not False
            and latent_attend_uses_tensor_cores(cache.dtype, C, R))
     if tensor_cores and not mma:
         raise ValueError("latent_attend: these shapes or dtypes do not run on the tensor cores")
+    part = None
+    if not mma or n_ranges > 1:
+        part = torch.empty(T * H * n_ranges * (C + 2), dtype=torch.float32, device=q_lat.device)
     if mma:
         n_req = req_start.numel() - 1
         max_tiles = -(-T * H // LATENT_MMA_ROWS) + n_req
         _check(lib().qb_latent_attend_mma(_p(q_lat), _p(q_rot), _p(cache), _p(part), _p(tok_pos), _p(req_start),
                                           _p(block_table), block_table.shape[1], n_req, T, H, C, R, page_size, num_pages,
-                                          int(n_ranges), max_tiles, ctypes.c_float(scale), _p(status), _stream()),
-               "latent_attend_mma")
+                                          int(n_ranges), max_tiles, int(window), int(float32_weights),
+                                          ctypes.c_float(scale), _p(sink), gate_p, gate_s, _p(out), _p(status),
+                                          _stream()), "latent_attend_mma")
+        if part is None:
+            return
     else:
         _check(lib().qb_latent_attend(_p(q_lat), _code(q_lat), _p(q_rot), _p(cache), _code(cache), _p(part), _p(tok_pos),
                                       _p(tok_req), _p(block_table), block_table.shape[1], T, H, C, R, page_size,
-                                      num_pages, int(n_ranges), ctypes.c_float(scale), _p(status), _stream()),
-               "latent_attend")
-    _check(lib().qb_latent_merge(_p(part), _p(sink), _p(out), _code(out), T, H, C, int(n_ranges), _stream()),
-           "latent_merge")
+                                      num_pages, int(n_ranges), int(window), ctypes.c_float(scale), _p(status),
+                                      _stream()), "latent_attend")
+    _check(lib().qb_latent_merge(_p(part), _p(sink), gate_p, gate_s, _p(out), _code(out), T, H, C, int(n_ranges),
+                                 _stream()), "latent_merge")
 
 
 # ---- sliding-window attention with extras (csrc/window_attention.cu) ---------------------------------------------
@@ -858,8 +897,9 @@ def window_attention_uses_tensor_cores(dtype, hd: int, vd: int) -> bool:
 def window_attention(q, k_cache, v_cache, out, tok_pos, tok_req, block_table, scale: float, window: int, status, *,
                      dist_bias=None, sink=None, softcap: float = 0.0, pool: int = 0, pooled_k=None, pooled_v=None,
                      pool_table=None, talk=None, scratch=None, n_split: int | None = None, n_requests: int | None = None,
-                     tensor_cores: bool | None = None) -> None:
-    """Softmax attention of every token over the last ``window`` keys of its request (0: all of them).  Options:
+                     tensor_cores: bool | None = None, chunk: int = 0) -> None:
+    """Softmax attention of every token over the last ``window`` keys of its request (0: all of them); ``chunk`` C > 0:
+    over the keys of its own chunk of C positions (counted from the request's first) only.  Options:
     ``dist_bias`` float32 ``[window, heads]`` added to the score by distance; ``sink`` float32 ``[heads]``, a term
     ``exp(sink)`` of the denominator; ``softcap`` c > 0: ``score <- c tanh(score / c)``; ``pool`` P with the pooled
     pages and their block table: one more key and value per block of P tokens that lies wholly before the window;
@@ -903,7 +943,7 @@ def window_attention(q, k_cache, v_cache, out, tok_pos, tok_req, block_table, sc
             _p(q), _code(q), _p(k_cache), _p(v_cache), _p(pooled_k), _p(pooled_v), _p(out), _p(scratch), _p(talk),
             _p(tok_pos), _p(tok_req), _p(block_table), block_table.shape[1], _p(pool_table),
             pool_table.shape[1] if pool_table is not None else 0, T, nq, nkv, hd, vd, page_size, num_pages, n_pool_pages,
-            ctypes.c_float(scale), ctypes.c_float(softcap), int(window), int(pool), _p(dist_bias), _p(sink), _p(status),
+            ctypes.c_float(scale), ctypes.c_float(softcap), int(window), int(pool), int(chunk), _p(dist_bias), _p(sink), _p(status),
             _stream()), "window_attention_mma", 1 + (talk is not None))
         return
     if n_split is None:
@@ -917,7 +957,7 @@ def window_attention(q, k_cache, v_cache, out, tok_pos, tok_req, block_table, sc
         _p(q), _code(q), _p(k_cache), _p(v_cache), _p(pooled_k), _p(pooled_v), _p(out), _p(scratch), _p(talk),
         _p(tok_pos), _p(tok_req), _p(block_table), block_table.shape[1], _p(pool_table),
         pool_table.shape[1] if pool_table is not None else 0, T, nq, nkv, hd, vd, page_size, num_pages, n_pool_pages,
-        ctypes.c_float(scale), ctypes.c_float(softcap), int(window), int(pool), _p(dist_bias), _p(sink), _p(part),
+        ctypes.c_float(scale), ctypes.c_float(softcap), int(window), int(pool), int(chunk), _p(dist_bias), _p(sink), _p(part),
         int(n_split), _p(status), _stream()), "window_attention", 1 + (talk is not None) + (n_split > 1))
 
 
@@ -1022,7 +1062,7 @@ def tanh_cap(x: torch.Tensor, cap: float) -> None:
     _check(lib().qb_tanh_cap(_p(x), ctypes.c_longlong(x.numel()), ctypes.c_float(cap), _stream()), "tanh_cap")
 
 
-GLU_SILU, GLU_CLAMPED = 0, 1
+GLU_SILU, GLU_CLAMPED, GLU_GELU_TANH = 0, 1, 2
 
 
 def glu_act(gate_up: torch.Tensor, out: torch.Tensor, *, bias=None, kind: int = GLU_SILU, limit: float = 0.0,
@@ -1030,7 +1070,7 @@ def glu_act(gate_up: torch.Tensor, out: torch.Tensor, *, bias=None, kind: int = 
     """The activation of a gated dense feed-forward from ``gate_up`` ``[n, 2 I]`` = ``[gate | up]`` (the activation
     dtype, or the product's float32 accumulators) into ``out`` ``[n, I]``; ``bias`` float32 ``[2 I]`` is added first.
     ``GLU_SILU``: ``silu(gate) * up``; ``GLU_CLAMPED``: ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``,
-    ``g * sigmoid(alpha * g) * (u + 1)``."""
+    ``g * sigmoid(alpha * g) * (u + 1)``; ``GLU_GELU_TANH``: ``gelu_tanh(gate) * up``."""
     n, two_i = gate_up.shape
     if tuple(out.shape) != (n, two_i // 2) or (gate_up.dtype != out.dtype and gate_up.dtype != torch.float32):
         raise ValueError("glu_act: shape/dtype mismatch")
@@ -1048,25 +1088,62 @@ GATED_DELTA_MAX_DIM = 256
 
 
 def gated_delta(qkv, ab, a_off: int, b_off: int, A_log, dt_bias, state, out, req_start, req_slot, n_heads: int,
-                n_groups: int, dim: int, vdim: int, q_scale: float, unit_eps: float) -> None:
+                n_groups: int, dim: int, vdim: int, q_scale: float, unit_eps: float, *, channel_decay=None) -> None:
     """The recurrence ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` per (request, head) over the
     step's tokens, from and into ``state`` ``[slots, heads, dim, vdim]`` float32.  ``qkv`` float32 ``[T, P]`` holds
     ``q | k`` (groups x dim each; head h reads group ``h // (heads / groups)``) and ``v`` (heads x vdim) in its
     first columns, after convolution and activation; q and k are made unit vectors per group here (``unit_eps``
     under the root), q also times ``q_scale``.  ``ab`` float32 rows whose columns ``a_off + h`` / ``b_off + h`` are
     the pre-activations of the decay ``g = exp(-exp(A_log) * softplus(a + dt_bias))`` and of ``beta = sigmoid(b)``.
-    ``out`` float32 ``[T, heads, vdim]``."""
+    ``out`` float32 ``[T, heads, vdim]``.  ``channel_decay`` (float32 ``[T, heads * dim]``, possibly a column range of
+    wider rows): the decay has one number per head and key channel, ``g = exp(-exp(A_log_h) * softplus(channel_decay +
+    dt_bias))`` with ``dt_bias`` ``[heads * dim]``, and row i of a head's S is multiplied by ``g_i``; ``a_off`` is not
+    read then."""
     for t, n in ((qkv, "qkv"), (ab, "ab"), (A_log, "A_log"), (dt_bias, "dt_bias"), (state, "state"), (out, "out")):
         _want(t, torch.float32, n)
     T = qkv.shape[0]
     H, G, D, DV = int(n_heads), int(n_groups), int(dim), int(vdim)
     if (qkv.stride(1) != 1 or ab.stride(1) != 1 or qkv.shape[1] < 2 * G * D + H * DV or ab.shape[0] != T
-            or min(a_off, b_off) < 0 or max(a_off, b_off) + H > ab.shape[1] or out.numel() != T * H * DV
-            or A_log.numel() != H or dt_bias.numel() != H or tuple(state.shape[1:]) != (H, D, DV) or H % G):
+            or b_off < 0 or b_off + H > ab.shape[1] or out.numel() != T * H * DV
+            or A_log.numel() != H or tuple(state.shape[1:]) != (H, D, DV) or H % G):
         raise ValueError("gated_delta: shape mismatch")
+    if channel_decay is None:
+        if a_off < 0 or a_off + H > ab.shape[1] or dt_bias.numel() != H:
+            raise ValueError("gated_delta: shape mismatch of the decay")
+        a_ptr, a_stride = ctypes.c_void_p(ab.data_ptr() + 4 * int(a_off)), int(ab.stride(0))
+    else:
+        a_ptr, a_stride = _rows_of(channel_decay, H * D, "channel_decay")
+        if channel_decay.shape[0] != T or dt_bias.numel() != H * D:
+            raise ValueError("gated_delta: shape mismatch of the decay")
     R = req_slot.numel()
-    scratch = torch.empty(T * (2 * G * D + 2 * H), dtype=torch.float32, device=qkv.device)
-    _check(lib().qb_gated_delta(ctypes.c_void_p(qkv.data_ptr()), int(qkv.stride(0)), ctypes.c_void_p(ab.data_ptr()),
-                                int(ab.stride(0)), int(a_off), int(b_off), _p(A_log), _p(dt_bias), _p(state), _p(out),
+    n_decay = H if channel_decay is None else H * D
+    scratch = torch.empty(T * (2 * G * D + n_decay + H), dtype=torch.float32, device=qkv.device)
+    _check(lib().qb_gated_delta(ctypes.c_void_p(qkv.data_ptr()), int(qkv.stride(0)), a_ptr, a_stride,
+                                ctypes.c_void_p(ab.data_ptr()), int(ab.stride(0)), int(b_off),
+                                int(channel_decay is not None), _p(A_log), _p(dt_bias), _p(state), _p(out),
                                 _p(scratch), _p(req_start), _p(req_slot), R, T, H, G, D, DV, ctypes.c_float(q_scale),
                                 ctypes.c_float(unit_eps), _stream()), "gated_delta", 2)
+
+
+# ---- a layer's input that belongs to the token itself (csrc/token_input.cu) --------------------------------------
+TOKEN_INPUT_SMALL = 32       # steps of at most this many tokens run the gate's product in the same launch
+
+
+def token_input(x, w_gate, table, offset: int, ids, out, status, gate=None) -> None:
+    """``out[t] = gelu_tanh(w_gate x_t) * table[ids[t], offset : offset + D]`` with ``w_gate`` ``[D, W]``.  ``gate``: the
+    product's float32 accumulators ``[T, D]`` when it was taken outside (``x`` is not read then); None: the product is
+    part of the launch.  ``table`` ``[vocab, >= offset + D]``."""
+    D, W = w_gate.shape
+    T = ids.numel()
+    _want(ids, torch.int32, "ids")
+    if tuple(out.shape) != (T, D) or table.dtype != out.dtype or offset < 0 or offset + D > table.shape[1]:
+        raise ValueError("token_input: shape/dtype mismatch")
+    if gate is not None:
+        g_p, g_s = _rows_of(gate, D, "gate")
+        _check(lib().qb_token_input_act(g_p, g_s, _p(table), table.shape[1], int(offset), _p(ids), _p(out), _code(out), T,
+                                        D, table.shape[0], _p(status), _stream()), "token_input_act")
+        return
+    if tuple(x.shape) != (T, W) or x.dtype != out.dtype or w_gate.dtype != out.dtype:
+        raise ValueError("token_input: shape/dtype mismatch")
+    _check(lib().qb_token_input_gate(_p(x), _p(w_gate), _p(table), table.shape[1], int(offset), _p(ids), _p(out),
+                                     _code(out), T, W, D, table.shape[0], _p(status), _stream()), "token_input_gate")

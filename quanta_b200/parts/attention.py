@@ -18,7 +18,10 @@ projected rows of a request are per-request state, so a portion that starts anyw
 sees); a learned number per q head that multiplies the head's scores (tensor ``names["head_temperature"]``
 ``[heads]``, float32; folded into the normed, rotated query); softmax weights that stay 32-bit on the tensor
 cores too (``float32_weights``: the kernels that feed ``P V`` with the weights in two bfloat16 parts, and float32
-arithmetic for single tokens, instead of the kernels that round the weights to bfloat16).
+arithmetic for single tokens, instead of the kernels that round the weights to bfloat16); values that are the projected
+keys themselves, before norm and rotation (``values_from_keys``: no ``v`` tensor); keys of the token's own chunk of the
+sequence only (``chunk``: position i sees j <= i with ``i // chunk == j // chunk``; with ``float32_weights``); the
+projection's float32 accumulators kept up to norm and rotation (``float32_projection``).
 """
 
 from __future__ import annotations
@@ -27,7 +30,7 @@ import torch
 
 from .. import kernels
 from ..matmul import empty_rows, linear
-from .base import CacheSpec, CacheStream, KeepAll, Mixer, TensorSpec, Window, make, register
+from .base import CacheSpec, CacheStream, KeepAll, Mixer, OwnChunk, TensorSpec, Window, make, register
 
 _NORM_KIND = {None: kernels.NORM_NONE, "per_layer": kernels.NORM_PER_LAYER, "per_head": kernels.NORM_PER_HEAD}
 
@@ -40,7 +43,8 @@ class GQAttention(Mixer):
                  position, qk_norm: str | None, qk_norm_eps: float, names: dict, window: int | None = None,
                  value_dim: int | None = None, q_temperature: tuple | None = None, own_kv: bool = True,
                  float32_output: bool = False, conv_taps: int = 0, conv_state_name: str = "attention_conv_inputs",
-                 float32_weights: bool = False):
+                 float32_weights: bool = False, values_from_keys: bool = False, chunk: int | None = None,
+                 float32_projection: bool = False):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} q heads are not a multiple of {n_kv_heads} kv heads")
         value_dim = head_dim if value_dim is None else int(value_dim)
@@ -63,7 +67,14 @@ class GQAttention(Mixer):
             raise ValueError("gqa_attention: the convolution on q, k, v needs keys and values of the layer's own and "
                              "no gate per head")
         self.conv_w = self.head_temp = None
-        self.float32_weights = bool(float32_weights)
+        self.float32_weights, self.float32_projection = bool(float32_weights), bool(float32_projection)
+        self.tied_v, self.chunk = bool(values_from_keys), None if chunk is None else int(chunk)
+        if self.tied_v and (self.vd != self.hd or not self.own_kv or self.taps):
+            raise ValueError("gqa_attention: values that are the keys have the keys' size and belong to a layer with keys "
+                             "of its own and no convolution")
+        if self.chunk is not None and (self.chunk < 1 or window is not None or not self.float32_weights):
+            raise ValueError("gqa_attention: a chunk holds at least one token, excludes a window, and is built into the "
+                             "kernels that keep the weights in 32 bits (float32_weights)")
         # the tensor-core kernels take equal key and value head sizes that are multiples of 16
         self.mma_shapes = self.hd == self.vd and self.hd % 16 == 0
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
@@ -78,7 +89,9 @@ class GQAttention(Mixer):
         n, H, hd, vd = self.names, self.hidden, self.hd, self.vd
         specs = [TensorSpec(n["q"], (self.nq * hd, H)), TensorSpec(n["o"], (H, self.nq * vd))]
         if self.own_kv:
-            specs += [TensorSpec(n["k"], (self.nkv * hd, H)), TensorSpec(n["v"], (self.nkv * vd, H))]
+            specs.append(TensorSpec(n["k"], (self.nkv * hd, H)))
+            if not self.tied_v:
+                specs.append(TensorSpec(n["v"], (self.nkv * vd, H)))
         if self.gated:
             specs.append(TensorSpec(n["g"], (self.nq, H)))
         if self.qk_norm is not None:
@@ -100,7 +113,7 @@ class GQAttention(Mixer):
         # padded to a multiple of 8 so that every row of the product starts on 16 bytes
         a = self.nq * self.hd
         b = a + (self.nkv * self.hd if self.own_kv else 0)
-        c = b + (self.nkv * self.vd if self.own_kv else 0)
+        c = b + (self.nkv * self.vd if self.own_kv and not self.tied_v else 0)
         self.gate_off = c
         rows = c + (self.nq if self.gated else 0)
         self.w_qkv = torch.zeros((-(-rows // 8) * 8, self.hidden), dtype=q.dtype, device=q.device)
@@ -108,7 +121,8 @@ class GQAttention(Mixer):
         del q
         if self.own_kv:
             self.w_qkv[a:b].copy_(fetch(n["k"]))
-            self.w_qkv[b:c].copy_(fetch(n["v"]))
+            if not self.tied_v:
+                self.w_qkv[b:c].copy_(fetch(n["v"]))
         if self.gated:
             self.w_qkv[c:rows].copy_(fetch(n["g"]))
         self.w_o = fetch(n["o"])
@@ -133,6 +147,7 @@ class GQAttention(Mixer):
         if not self.own_kv:
             return None
         return CacheSpec((CacheStream("k", self.nkv, self.hd), CacheStream("v", self.nkv, self.vd)),
+                         OwnChunk(self.chunk) if self.chunk is not None else
                          KeepAll() if self.window is None else Window(int(self.window)))
 
     def forward(self, x, ctx, cache, state):
@@ -146,7 +161,7 @@ class GQAttention(Mixer):
                 torch.empty((0, 0, C), dtype=torch.float32, device=x.device)
             kernels.short_conv(proj[:, :C], self.conv_w, hist, qkv, ctx.tok_req, ctx.req_start, ctx.req_slot, plain=True)
         else:
-            qkv = linear(x, self.w_qkv)
+            qkv = linear(x, self.w_qkv, out_dtype=torch.float32 if self.float32_projection else None)
         q = torch.empty((T, self.nq, self.hd), dtype=x.dtype, device=x.device)
         tables = self.position.rotary_tables(x.device)
         if tables is None:
@@ -168,7 +183,8 @@ class GQAttention(Mixer):
             self.k_norm_w, _NORM_KIND[self.qk_norm], self.eps, inv_freq, pair_axis, ctx.positions, ctx.tok_pos,
             ctx.tok_req, cache.block_table, self.nq, self.nkv, self.hd, rd, cache.page_size, ctx.status,
             vd=self.vd, has_kv=self.own_kv, q_temp_coef=self.q_temp[0], q_temp_every=self.q_temp[1],
-            head_scale=self.head_temp)
+            head_scale=self.head_temp, interleaved=bool(getattr(self.position, "interleaved", False)),
+            tied_values=self.tied_v)
         out = empty_rows(T, self.nq, self.vd, dtype=x.dtype, device=x.device)
         self.attend(q, cache, out, ctx)
         if self.gated:
@@ -190,9 +206,10 @@ class GQAttention(Mixer):
             # about 2,048 warps in all, at least 32 keys a range (measured on a B200 with 4 kv heads of 128: 8 tokens
             # over 2,048 keys 47 us with 64 ranges against 63 with 32; 32 tokens 120 us with 16 against 150 with 64; one
             # token over 8,192 keys 61 us with 256 against 110 with 64)
-            n_split = max(1, min(-(-2048 // warps), -(-max(1, ctx.max_len_after) // 32), 256))
+            keys = max(1, min(ctx.max_len_after, self.chunk or self.window or ctx.max_len_after))
+            n_split = max(1, min(-(-2048 // warps), -(-keys // 32), 256))
             kernels.window_attention(q, cache.k, cache.v, out, ctx.tok_pos, ctx.tok_req, cache.block_table, self.scale,
-                                     window, ctx.status, n_split=n_split, n_requests=R)
+                                     window, ctx.status, n_split=n_split, n_requests=R, chunk=self.chunk or 0)
             return
         if q.dtype != torch.bfloat16 or not self.mma_shapes:
             kernels.paged_attention_simt(q, cache.k, cache.v, out, ctx.tok_pos, ctx.tok_req, cache.block_table,

@@ -1,8 +1,9 @@
 """What a part is, and the registries parts are chosen from.
 
-A model is put together from parts of eight kinds: ``mixer`` (attention, or a recurrence with a state
+A model is put together from parts of nine kinds: ``mixer`` (attention, or a recurrence with a state
 of fixed size), ``feed_forward`` (dense or routed experts), ``norm``, ``position`` (position encoding),
-``time_conv`` (a short convolution over time in front of a sublayer), ``block`` (how a layer arranges
+``time_conv`` (a short convolution over time in front of a sublayer), ``token_input`` (what a layer adds
+for the token itself, whatever its context), ``block`` (how a layer arranges
 the others), ``embedding`` (token ids to the residual stream) and ``head`` (the residual stream to
 logits).  A part takes every size and constant as a constructor parameter, names
 the checkpoint tensors it needs (``tensor_specs``), receives them (``load``) and runs on the tokens
@@ -20,7 +21,7 @@ from typing import Any, Callable
 
 import torch
 
-KINDS = ("mixer", "feed_forward", "norm", "position", "time_conv", "block", "embedding", "head")
+KINDS = ("mixer", "feed_forward", "norm", "position", "time_conv", "token_input", "block", "embedding", "head")
 _REGISTRY: dict[str, dict[str, type]] = {k: {} for k in KINDS}
 
 
@@ -114,6 +115,16 @@ class WindowAndOpenBlock(Retention):
 
 
 @dataclass(frozen=True)
+class OwnChunk(Retention):
+    """A query at position p reads the keys of its own chunk only, ``floor(p / chunk) * chunk .. p``; chunks are counted
+    from position 0."""
+    chunk: int = 1
+
+    def needed_ranges(self, length):
+        return [(length // self.chunk * self.chunk, None)]
+
+
+@dataclass(frozen=True)
 class CacheSpec:
     """A mixer's need of paged per-token storage: its streams and what is retained.  Layers with equal
     specs form one group of the cache manager: they share pages ids and block tables.  ``stride`` > 1: the
@@ -188,6 +199,7 @@ class StepContext:
     dec_tok: torch.Tensor | None = None        # int32 [n_dec] token rows (device)
     n_dec: int = 0
     spans: list | None = None
+    token_ids: torch.Tensor | None = None      # int32 [T] the step's token ids (set by the model)
     work: dict = field(default_factory=dict)   # per-step scratch shared by the layers (tile lists and the like)
 
 
@@ -371,6 +383,14 @@ class TimeConv(Part):
         return {}
 
     def forward(self, x: torch.Tensor, ctx: StepContext, state: dict[str, torch.Tensor], out: torch.Tensor) -> None:
+        raise NotImplementedError
+
+
+class TokenInput(Part):
+    """What a layer adds to the residual stream for the token itself: ``forward(x [T, hidden] in the activation dtype,
+    ctx) -> pending contribution`` reads the stream's copy ``x`` and the token ids of the step (``ctx.token_ids``)."""
+
+    def forward(self, x: torch.Tensor, ctx: StepContext):
         raise NotImplementedError
 
 

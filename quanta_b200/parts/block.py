@@ -12,7 +12,8 @@ import torch
 from .. import kernels
 from ..matmul import empty_rows, linear
 from . import norms as _norms
-from .base import Addends, Block, Embedding, Head, NormedPending, StreamCopy, StreamsPending, TensorSpec, make, register
+from .base import (Addends, Block, Embedding, Head, NormedPending, StreamCopy, StreamsPending, TensorSpec, make, register,
+                   run_beside)
 
 
 @register("block", "pre_norm")
@@ -104,6 +105,53 @@ class SandwichNormBlock(Block):
         x2 = empty_rows(T, self.hidden, dtype=ctx.dtype, device=h.device)
         self.feed_forward_norm.forward(h, d, x2)
         return NormedPending(self.feed_forward.forward(x2, ctx), self.feed_forward_post_norm)
+
+
+@register("block", "parallel_residual")
+class ParallelBlock(Block):
+    """Mixer and feed-forward read ONE norm of the stream and join it together, ``h += mixer(norm(h)) +
+    feed_forward(norm(h))`` (the feed-forward is optional); then, where the layer has one, the token's own input
+    (a ``token_input`` part) reads the new stream and stays pending.  The two sublayers share nothing but their input,
+    so the feed-forward runs on a second CUDA stream beside the mixer; their float32 outputs, the stream's sum and its
+    copy for the token input are one launch."""
+
+    graph_safe = True
+
+    def __init__(self, hidden_size: int, mixer, norm, feed_forward=None, token_input=None):
+        self.hidden = int(hidden_size)
+        self.mixer = make("mixer", mixer)
+        self.norm = make("norm", norm)
+        self.feed_forward = make("feed_forward", feed_forward) if feed_forward is not None else None
+        self.token_input = make("token_input", token_input) if token_input is not None else None
+
+    def children(self):
+        return [p for p in (self.norm, self.mixer, self.feed_forward, self.token_input) if p is not None]
+
+    def forward(self, h, pending, ctx, cache, state):
+        T = h.shape[0]
+        x = empty_rows(T, self.hidden, dtype=ctx.dtype, device=h.device)
+        self.norm.forward(h, pending, x)
+        if self.feed_forward is None:
+            total = self.mixer.forward(x, ctx, cache, state)
+            total = total if isinstance(total, Addends) else Addends(_float32(total))
+        else:
+            f, m = run_beside(lambda: self.feed_forward.forward(x, ctx),
+                              lambda: self.mixer.forward(x, ctx, cache, state), h.device)
+            if isinstance(f, Addends) or isinstance(m, Addends):
+                raise NotImplementedError("parallel_residual: sublayers whose output is itself an untaken sum")
+            f, m = _float32(f), _float32(m)
+            if f.dim() == 3 and m.dim() == 3:
+                raise NotImplementedError("parallel_residual: slots in both sublayers' outputs")
+            total = Addends(m, extra=f) if f.dim() == 2 else Addends(f, extra=m)
+        if self.token_input is None:
+            return total
+        x2 = empty_rows(T, self.hidden, dtype=ctx.dtype, device=h.device)
+        _norms.add_sum(h, total, x2)
+        return self.token_input.forward(x2, ctx)
+
+
+def _float32(y):
+    return y if y.dtype == torch.float32 else y.float()
 
 
 @register("block", "hyper_connected")

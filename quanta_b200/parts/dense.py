@@ -1,6 +1,6 @@
 """Dense feed-forwards: gated, ``down(act(gate x) * (up x))`` with ``act = silu`` (optionally with a bias on each of
 the three projections), or in the clamped form ``g = min(gate x, limit)``, ``u = clamp(up x, -limit, limit)``,
-``down(g * sigmoid(alpha g) * (u + 1))``; and ungated, ``down(act(up x))`` with ``act`` the square of relu.
+``down(g * sigmoid(alpha g) * (u + 1))``, or with the tanh form of gelu for silu; and ungated, ``down(act(up x))`` with ``act`` the square of relu.
 
 The gate and up matrices are held as one, so a step is two library products and one activation kernel.
 The result is float32 (the accumulator of the down product), for blocks that norm it before the sum.
@@ -18,14 +18,15 @@ from .base import Addends, FeedForward, TensorSpec, register
 @register("feed_forward", "gated_dense")
 class GatedDense(FeedForward):
     graph_safe = True
+    KINDS = {"silu": kernels.GLU_SILU, "clamped": kernels.GLU_CLAMPED, "gelu_tanh": kernels.GLU_GELU_TANH}
 
     def __init__(self, hidden_size: int, inner_size: int, names: dict, activation: str = "silu", biases: bool = False,
                  limit: float = 0.0, alpha: float = 1.0):
         """``names``: gate, up, down, and with ``biases`` gate_b, up_b, down_b (float32 vectors; the down bias is
-        handed on as an addend of the output, for the norm kernel that reads it).  ``activation``: ``"silu"`` or
-        ``"clamped"`` (with ``limit`` and ``alpha``)."""
-        if activation not in ("silu", "clamped"):
-            raise ValueError(f"gated_dense: activation {activation!r} is not built (silu and clamped are)")
+        handed on as an addend of the output, for the norm kernel that reads it).  ``activation``: ``"silu"``,
+        ``"gelu_tanh"`` or ``"clamped"`` (with ``limit`` and ``alpha``)."""
+        if activation not in self.KINDS:
+            raise ValueError(f"gated_dense: activation {activation!r} is not built ({', '.join(self.KINDS)} are)")
         if activation == "clamped" and not limit > 0:
             raise ValueError(f"gated_dense: the clamped activation needs a positive limit, got {limit}")
         self.hidden, self.inner, self.names = int(hidden_size), int(inner_size), dict(names)
@@ -60,7 +61,7 @@ class GatedDense(FeedForward):
             kernels.silu_mul(gate_up, act)
         else:
             kernels.glu_act(gate_up, act, bias=self.b_gate_up, limit=self.limit, alpha=self.alpha,
-                            kind=kernels.GLU_CLAMPED if self.activation == "clamped" else kernels.GLU_SILU)
+                            kind=self.KINDS[self.activation])
         y = linear(act, self.w_down, out_dtype=torch.float32)
         return Addends(y, bias=self.b_down) if self.biases else y
 

@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
-from .base import Norm, NormedPending, StreamCopy, StreamsPending, TensorSpec, register
+from .base import Addends, Norm, NormedPending, StreamCopy, StreamsPending, TensorSpec, register
 
 
 @register("norm", "rms_norm")
@@ -58,6 +58,10 @@ class RMSNorm(Norm):
                 normed_add(h, delta, self.weight, self.eps, out, rows, store_h, groups=self.groups)
                 return
             delta = delta.materialize()
+        if isinstance(delta, Addends):
+            # a sum that nobody has taken yet joins the stream as it is
+            add_sum(h, delta, out, weight=self.weight, groups=self.groups, eps=self.eps, rows=rows, store_h=store_h)
+            return
         if self.groups != 1:
             if delta is not None and delta.dtype != torch.float32:
                 delta = delta.float()
@@ -87,6 +91,14 @@ def normed_add(h, delta: NormedPending, weight, eps: float, out, rows, store_h: 
                                extra_bias=a.extra_bias)
 
 
+def add_sum(h, a: Addends, out, weight=None, groups: int = 1, eps: float = 0.0, rows=None, store_h: bool = True) -> None:
+    """``h += the sum of a`` and ``out = weight * rms(h)`` (``weight`` None: ``out = h`` in out's dtype) in one launch."""
+    kernels.grouped_normed_add(h, y=a.y, y_scale=a.scale, y_bias=a.bias, y_gain=a.y_gain, extra=a.extra,
+                               extra_scale=a.extra_scale, extra_bias=a.extra_bias, extra_gain=a.extra_gain,
+                               branch_eps=a.branch_eps, weight=weight, weight_groups=groups, eps=eps, out=out, rows=rows,
+                               store_h=store_h)
+
+
 @register("norm", "none")
 class NoNorm(Norm):
     """No norm: the sublayer reads the residual stream as it is.  ``forward`` still takes the pending contribution
@@ -108,6 +120,9 @@ class NoNorm(Norm):
             return
         if isinstance(delta, NormedPending):
             delta = delta.materialize()
+        if isinstance(delta, Addends):
+            add_sum(h, delta, out, rows=rows, store_h=store_h)
+            return
         if delta is not None:
             kernels.residual_add(h, delta)
         kernels.normed_add_rmsnorm(h, None, None, 0.0, None, 0.0, out, rows=rows, store_h=False)

@@ -10,6 +10,10 @@ one position to every axis, so the numbers equal the unsectioned ladder.
 frequency whose wavelength is shorter than ``original / high`` is kept, one longer than ``original / low`` is
 divided by ``factor``, and between the two, with ``s = (original / l - low) / (high - low)``, it becomes
 ``(1 - s) f / factor + s f``.
+
+``interleaved``: the rotated pairs are neighbours, ``(2j, 2j + 1)``, instead of ``(j, j + rotary_dim/2)`` (the mixers
+hand this to the kernels that rotate).  ``float64_ladder``: the ladder is computed in float64 and rounded once, as it
+always is with ``wavelength_scaling``.
 """
 
 from __future__ import annotations
@@ -25,7 +29,8 @@ from .base import PositionEncoding, register
 class PartialRotary(PositionEncoding):
     graph_safe = True
 
-    def __init__(self, head_dim: int, rotary_dim: int, theta: float, sections=None, wavelength_scaling=None):
+    def __init__(self, head_dim: int, rotary_dim: int, theta: float, sections=None, wavelength_scaling=None,
+                 interleaved: bool = False, float64_ladder: bool = False):
         if rotary_dim % 2 or not 0 <= rotary_dim <= head_dim:
             raise ValueError(f"rotary_dim {rotary_dim} must be even and at most head_dim {head_dim}")
         if sections is not None and sum(sections) != rotary_dim // 2:
@@ -33,6 +38,7 @@ class PartialRotary(PositionEncoding):
         self.head_dim, self.rotary_dim, self.theta = int(head_dim), int(rotary_dim), float(theta)
         self.sections = None if sections is None else tuple(int(s) for s in sections)
         self.n_axes = 1 if self.sections is None else len(self.sections)
+        self.interleaved, self.float64_ladder = bool(interleaved), bool(float64_ladder)
         self.wavelength_scaling = None
         if wavelength_scaling is not None:
             factor, low, high, original = (float(v) for v in wavelength_scaling)
@@ -44,10 +50,12 @@ class PartialRotary(PositionEncoding):
 
     def inv_freq(self) -> torch.Tensor:
         rd = self.rotary_dim
-        if self.wavelength_scaling is None:
+        if self.wavelength_scaling is None and not self.float64_ladder:
             return 1.0 / (self.theta ** (torch.arange(0, rd, 2, dtype=torch.float32) / rd))
         # the ladder and its rescaling in float64, rounded once to the float32 the kernels multiply positions with
         f = self.theta ** (-torch.arange(0, rd, 2, dtype=torch.float64) / rd)
+        if self.wavelength_scaling is None:
+            return f.to(torch.float32)
         factor, low, high, original = self.wavelength_scaling
         wavelength = 2.0 * math.pi / f
         s = ((original / wavelength - low) / (high - low)).clamp(0.0, 1.0)

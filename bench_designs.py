@@ -1,4 +1,4 @@
-"""``bench.py --design guravik`` / ``--design tirizen`` / ``--design tarulix`` / ``--design puvolix``: another decoder beside the MiniMax-M3 decoder at equal sizes.
+"""``bench.py --design guravik`` / ``--design tirizen`` / ``--design tarulix`` / ``--design puvolix`` / ``--design lotilix``: another decoder beside the MiniMax-M3 decoder at equal sizes.
 
 For a few sizes that resemble a real model's layers (seeded random weights, bfloat16): one prompt of
 ``--prompt-len`` tokens as one step (tokens a second) and decode steps of ``--batch`` requests at that
@@ -34,6 +34,14 @@ shared experts), and MiniMax-M3, all at equal sizes.  Alone: the attention kerne
 (no window) beside Tarulix's biased form and MiniMax-M3's; ``gated_delta`` beside Guravik's ``delta_rule`` (the like
 chain in time) and Tirizen's ``gla``; the launch between two sublayers (``grouped_normed_add`` with branch norms,
 and with the depth-weighted sum) beside ``normed_add_rmsnorm``.
+
+``--design lotilix``: the Lotilix decoder (layers: windowed latent attention with gates, a gated delta rule with a decay
+per key channel, chunked attention whose values are its keys; a dense feed-forward beside each mixer; a gated row of the
+token's own in every layer) beside Guravik, the closest existing model (latent attention, a delta rule with a decay per
+channel, dense feed-forwards; given a feed-forward in every layer here), and MiniMax-M3, all at equal sizes.  Alone: the
+latent attention beside Guravik's form of it, the chunked attention beside Puvolix's form of the same kernels, the
+recurrence beside Puvolix's (one decay a head) and Guravik's ``delta_rule``, and the launches around the token's own input
+beside ``normed_add_rmsnorm``.
 """
 
 from __future__ import annotations
@@ -149,6 +157,42 @@ def minimax_raw(s: dict) -> dict:
                 model_type="minimax_m3")
 
 
+LOTILIX_SIZES = {
+    "w2048": dict(width=2048, groups=2, vocab=32000, ff=5632, attn_heads=16, dim=128, rot=64, vdim=128, q_rank=768, kv_rank=256,
+                  window=1024, chunk=1024, delta_heads=16, delta_dim=128, inner_rank=128, side=256),
+    "w4096": dict(width=4096, groups=2, vocab=32000, ff=11008, attn_heads=32, dim=128, rot=64, vdim=128, q_rank=1536, kv_rank=512,
+                  window=1024, chunk=1024, delta_heads=32, delta_dim=128, inner_rank=128, side=256),
+}
+
+
+def lotilix_raw(s: dict) -> dict:
+    """Per group of three layers: windowed latent attention, the gated delta rule (heads of 128 x 128, convolutions of 4
+    taps), chunked attention (a quarter as many kv heads); every layer with a dense feed-forward and a token row."""
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    latent = {"heads": s["attn_heads"], "dim": s["dim"], "rot_dim": s["rot"], "vdim": s["vdim"], "q_rank": s["q_rank"],
+              "kv_rank": s["kv_rank"], "scale": 1.0 / math.sqrt(s["dim"] + s["rot"]), "mask": {"size": s["window"]},
+              "rot": {"base": 1e6, "dims": s["rot"]}}
+    delta = {"heads": s["delta_heads"], "kv_heads": s["delta_heads"], "dim": s["delta_dim"], "vdim": s["delta_dim"], "conv": 4,
+             "decay_rank": s["inner_rank"], "gate_rank": s["inner_rank"]}
+    attn = {"heads": s["attn_heads"], "kv_heads": max(1, s["attn_heads"] // 4), "dim": s["dim"], "vdim": s["dim"],
+            "scale": 1.0 / math.sqrt(s["dim"]), "mask": {"size": s["chunk"]},
+            "rot": {"dims": s["dim"], "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    layers = [{"type": "latent_attention", "mixer": latent, "mlp": mlp}, {"type": "channel_delta", "mixer": delta, "mlp": mlp},
+              {"type": "attention", "mixer": attn, "mlp": mlp}] * s["groups"]
+    return {"architecture": "Lotilix", "vocab": s["vocab"], "width": s["width"], "layers": layers, "norm": {"eps": 1e-5},
+            "token_side": {"dim": s["side"]}}
+
+
+def guravik_like_lotilix_raw(s: dict) -> dict:
+    """Guravik with as many layers and a feed-forward in each: latent attention, delta rule, latent attention."""
+    raw = guravik_raw(dict(s))
+    for layer in raw["layers"]:
+        layer["mlp"] = {"kind": "dense", "ff": s["ff"]}
+    for i in range(2, len(raw["layers"]), 3):
+        raw["layers"][i] = raw["layers"][i - 2]
+    return raw
+
+
 def _model_numbers(cfg, prompt_len: int, batch: int, steps: int, warmup: int) -> dict:
     import torch
     from quanta_b200 import kernels
@@ -199,7 +243,8 @@ def _model_numbers(cfg, prompt_len: int, batch: int, steps: int, warmup: int) ->
 
 
 # ---- kernels alone -------------------------------------------------------------------------------------
-def latent_prefill(tokens: int, heads: int, C: int, R: int, page: int = 16) -> dict:
+def latent_prefill(tokens: int, heads: int, C: int, R: int, page: int = 16, window: int = 0, lotilix: bool = False) -> dict:
+    """``lotilix``: with gates and 32-bit softmax weights instead of a sink."""
     import torch
     import bench_kernels as bk
     from quanta_b200 import kernels as k
@@ -215,14 +260,17 @@ def latent_prefill(tokens: int, heads: int, C: int, R: int, page: int = 16) -> d
     req = torch.zeros(tokens, dtype=torch.int32, device=dev)
     st = k.new_status(dev)
     starts = torch.tensor([0, tokens], dtype=torch.int32, device=dev)
-    ms = bk.timed(lambda: k.latent_attend(q_lat, q_rot, cache, sink, out, pos, req, table, 0.1, 1, st, req_start=starts), n=5, warm=2)
-    keys = tokens * (tokens + 1) // 2
+    opts = dict(gate=torch.randn(tokens, heads, device=dev), float32_weights=True) if lotilix else {}
+    ms = bk.timed(lambda: k.latent_attend(q_lat, q_rot, cache, None if lotilix else sink, out, pos, req, table, 0.1, 1, st,
+                                          req_start=starts, window=window, **opts), n=5, warm=2)
+    keys = sum(min(p + 1, window or p + 1) for p in range(tokens))
     flops = (2.0 * (C + R) + 2.0 * C) * heads * keys
     return {"kernel": "latent_attend (prompt)", "tokens": tokens, "heads": heads, "latent": C, "rot": R, "ms": round(ms, 3),
             "TFLOP/s": round(flops / ms / 1e9, 2)}
 
 
-def latent_decode(batch: int, context: int, heads: int, C: int, R: int, page: int = 16) -> dict:
+def latent_decode(batch: int, context: int, heads: int, C: int, R: int, page: int = 16, window: int = 0,
+                  lotilix: bool = False) -> dict:
     import torch
     import bench_kernels as bk
     from quanta_b200 import kernels as k
@@ -239,16 +287,19 @@ def latent_decode(batch: int, context: int, heads: int, C: int, R: int, page: in
     req = torch.arange(batch, dtype=torch.int32, device=dev)
     st = k.new_status(dev)
     blocks = -(-batch * heads // k.LATENT_MMA_ROWS) if k.latent_attend_uses_tensor_cores(torch.bfloat16, C, R) else batch * -(-heads // 8)
-    n_ranges = max(1, min(64, -(-296 // blocks), -(-context // 128)))
+    seen = min(context, window + k.LATENT_MMA_ROWS) if window else context
+    n_ranges = max(1, min(64, -(-296 // blocks), -(-seen // 128)))
+    opts = dict(gate=torch.randn(batch, heads, device=dev), float32_weights=True) if lotilix else {}
     starts = torch.arange(batch + 1, dtype=torch.int32, device=dev)
 
     def all_layers():
         for c in caches:
-            k.latent_attend(q_lat, q_rot, c, sink, out, pos, req, table, 0.1, n_ranges, st, req_start=starts)
+            k.latent_attend(q_lat, q_rot, c, None if lotilix else sink, out, pos, req, table, 0.1, n_ranges, st, req_start=starts,
+                            window=window, **opts)
     ms = bk.timed_graph(all_layers, reps=1) / layers
-    nbytes = batch * context * (C + R) * 2
+    nbytes = batch * min(context, window or context) * (C + R) * 2
     return {"kernel": "latent_attend + merge (single tokens)", "batch": batch, "context": context, "heads": heads, "latent": C,
-            "rot": R, "ranges": n_ranges, "us": round(ms * 1e3, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
+            "rot": R, "window": window, "ranges": n_ranges, "us": round(ms * 1e3, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
 
 
 def delta_rule(tokens_per_req: int, reqs: int, heads: int, D: int) -> dict:
@@ -417,10 +468,11 @@ def window_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int,
             "TFLOP/s": round(flops / ms / 1e9, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
 
 
-def plain_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int, hd: int, page: int = 16) -> dict:
+def plain_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int, hd: int, page: int = 16, chunk: int = 0) -> dict:
     """The attention as Puvolix runs it: ``window_attention`` over all keys, no extras; portions on the tensor cores
     with the weights in two bfloat16 parts, single tokens with their keys cut into ranges and a join (32-bit
-    arithmetic).  Flops count ``4 * head_dim`` a (query head, visible key); bytes the visible keys and values once."""
+    arithmetic); ``chunk``: only the keys of the token's own chunk, as Lotilix runs it.  Flops count ``4 * head_dim`` a
+    (query head, visible key); bytes the visible keys and values once."""
     import torch
     import bench_kernels as bk
     from quanta_b200 import kernels as k
@@ -437,24 +489,26 @@ def plain_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int, 
     pos = torch.arange(context - tokens_per_req, context, dtype=torch.int32, device=dev).repeat(reqs)
     req = torch.arange(reqs, dtype=torch.int32, device=dev).repeat_interleave(tokens_per_req)
     st = k.new_status(dev)
-    n_split = max(1, min(-(-2048 // (T * nkv)), -(-context // 32), 256))      # as parts/attention.py chooses it
+    n_split = max(1, min(-(-2048 // (T * nkv)), -(-min(context, chunk or context) // 32), 256))      # as parts/attention.py
 
     def all_layers():
         for kc, vc in caches:
-            k.window_attention(q, kc, vc, out, pos, req, table, hd ** -0.5, 0, st, n_split=n_split, n_requests=reqs)
+            k.window_attention(q, kc, vc, out, pos, req, table, hd ** -0.5, 0, st, n_split=n_split, n_requests=reqs, chunk=chunk)
     ms = (bk.timed_graph(all_layers, reps=1) if single else bk.timed(all_layers, n=5, warm=2)) / layers
     k.raise_on_status(st.cpu())
-    seen = sum(p_ + 1 for p_ in range(context - tokens_per_req, context))
+    seen = sum(p_ + 1 - (p_ // chunk * chunk if chunk else 0) for p_ in range(context - tokens_per_req, context))
     flops = 4.0 * hd * nq * seen * reqs
-    nbytes = reqs * context * nkv * hd * 2 * 2
-    return {"kernel": "window_attention (all keys, no extras)", "requests": reqs, "tokens_per_request": tokens_per_req,
+    first = (context - tokens_per_req) // chunk * chunk if chunk else 0
+    nbytes = reqs * (context - first) * nkv * hd * 2 * 2
+    return {"kernel": "window_attention (own chunk)" if chunk else "window_attention (all keys, no extras)", "chunk": chunk, "requests": reqs, "tokens_per_request": tokens_per_req,
             "context": context, "q_heads": nq, "kv_heads": nkv, "head_dim": hd, "layers": layers, "ranges": n_split if single else 1,
             "us": round(ms * 1e3, 2), "TFLOP/s": round(flops / ms / 1e9, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
 
 
-def gated_delta(tokens_per_req: int, reqs: int, heads: int, groups: int, D: int, DV: int) -> dict:
+def gated_delta(tokens_per_req: int, reqs: int, heads: int, groups: int, D: int, DV: int, channel: bool = False) -> dict:
     """``gated_delta`` alone (preparation + chain).  Bytes: the state read and written, and per token the rows read
-    (q, k, v, the two pre-activations), the unit q and k written and read, and the output."""
+    (q, k, v, the two pre-activations), the unit q and k written and read, and the output; ``channel``: a decay per key
+    channel (its pre-activations read, the decays written and read)."""
     import torch
     import bench_kernels as bk
     from quanta_b200 import kernels as k
@@ -463,7 +517,8 @@ def gated_delta(tokens_per_req: int, reqs: int, heads: int, groups: int, D: int,
     C = 2 * groups * D + heads * DV
     qkv = torch.randn(T, C, device=dev)
     ab = torch.randn(T, 2 * heads, device=dev)
-    A_log, dt_b = torch.zeros(heads, device=dev), torch.zeros(heads, device=dev)
+    A_log, dt_b = torch.zeros(heads, device=dev), torch.zeros(heads * (D if channel else 1), device=dev)
+    decay = torch.randn(T, heads * D, device=dev) if channel else None
     layers = 1 if tokens_per_req > 1 else max(1, min(16, int(2e9 // (reqs * heads * D * DV * 4))))
     states = [torch.zeros(reqs, heads, D, DV, device=dev) for _ in range(layers)]
     out = torch.empty(T, heads, DV, device=dev)
@@ -472,10 +527,13 @@ def gated_delta(tokens_per_req: int, reqs: int, heads: int, groups: int, D: int,
 
     def all_layers():
         for s in states:
-            k.gated_delta(qkv, ab, 0, heads, A_log, dt_b, s, out, starts, slots, heads, groups, D, DV, D ** -0.5, 1e-6)
+            k.gated_delta(qkv, ab, 0, heads, A_log, dt_b, s, out, starts, slots, heads, groups, D, DV, D ** -0.5, 1e-6,
+                          channel_decay=decay)
     ms = (bk.timed_graph(all_layers, reps=1) if tokens_per_req == 1 else bk.timed(all_layers, n=5, warm=2)) / layers
     nbytes = 2 * reqs * heads * D * DV * 4 + T * (C + 2 * heads + 4 * groups * D + heads * DV) * 4
-    return {"kernel": "gated_delta (preparation + chain)", "requests": reqs, "tokens_per_request": tokens_per_req, "heads": heads,
+    if channel:
+        nbytes += T * (3 * heads * D - heads) * 4
+    return {"kernel": "gated_delta (preparation + chain)", "decay": "channel" if channel else "head", "requests": reqs, "tokens_per_request": tokens_per_req, "heads": heads,
             "groups": groups, "dim": D, "value_dim": DV, "layers": layers, "us": round(ms * 1e3, 2),
             "tokens/s": round(T / ms * 1e3, 1), "GB/s": round(nbytes / ms / 1e6, 1),
             "fp32 TFLOP/s": round(7.0 * D * DV * heads * T / ms / 1e9, 2)}
@@ -511,6 +569,94 @@ def between_sublayers(tokens: int, H: int, groups: int, depth: int) -> dict:
     for name, ms in (("branches + group norm", t_mix), ("slots + shared + depth sum", t_depth), ("normed_add_rmsnorm", t_old)):
         res[name] = {"us": round(ms * 1e3, 2), "GB/s": round(by[name] / ms / 1e6, 1)}
     return res
+
+
+def token_input(tokens: int, H: int, D: int, vocab: int = 32000) -> dict:
+    """The launches around a token's own input: the sum of both sublayers' outputs into the stream with its bfloat16
+    copy (``grouped_normed_add``), the gate (one launch in steps of few tokens, a library product and the activation
+    else), the projection (a library product) with the norm, sum and next norm (``normed_add_rmsnorm``)."""
+    import torch
+    import bench_kernels as bk
+    from quanta_b200 import kernels as k
+    from quanta_b200.matmul import linear
+    dev = bk.DEV
+    h, a, b, y = (torch.randn(tokens, H, device=dev) for _ in range(4))
+    x = torch.randn(tokens, H, device=dev).to(torch.bfloat16)
+    out = torch.empty(tokens, H, device=dev, dtype=torch.bfloat16)
+    g1, w = torch.ones(H, device=dev), torch.ones(H, device=dev)
+    table = torch.randn(vocab, 4 * D, device=dev).to(torch.bfloat16)
+    wg = torch.randn(D, H, device=dev).to(torch.bfloat16)
+    ids = torch.randint(0, vocab, (tokens,), dtype=torch.int32, device=dev)
+    g = torch.empty(tokens, D, device=dev, dtype=torch.bfloat16)
+    st = k.new_status(dev)
+    small = tokens <= k.TOKEN_INPUT_SMALL
+    run = (lambda f: bk.timed_graph(f, reps=20)) if tokens <= 64 else (lambda f: bk.timed(f, n=10, warm=3))
+    t_sum = run(lambda: k.grouped_normed_add(h, y=a, extra=b, out=out))
+    t_gate = run(lambda: k.token_input(x, wg, table, D, ids, g, st, gate=None if small else linear(x, wg, out_dtype=torch.float32)))
+    t_norm = run(lambda: k.normed_add_rmsnorm(h, y, g1, 1e-5, w, 1e-5, out))
+    row = H * 4
+    res = {"tokens": tokens, "width": H, "dim": D}
+    for name, ms, nbytes in (("sum + copy", t_sum, tokens * (4 * row + H * 2)),
+                             ("gate", t_gate, tokens * (H + 2 * D) * 2 + D * H * 2 + (0 if small else tokens * D * 8)),
+                             ("normed_add_rmsnorm", t_norm, tokens * (3 * row + H * 2))):
+        res[name] = {"us": round(ms * 1e3, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
+    return res
+
+
+def run_lotilix(args) -> dict:
+    import bench
+    from quanta_b200.config import GuravikConfig, LotilixConfig, MiniMaxM3Config
+    pk, pk_src = bench.peaks()
+    clocks = bench.ClockSampler()
+    clocks.start()
+    models = {}
+    for name, s in LOTILIX_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        t0 = time.time()
+        p = _model_numbers(LotilixConfig.from_dict(lotilix_raw(s)), args.prompt_len, args.batch, args.steps, args.warmup)
+        g = _model_numbers(GuravikConfig.from_dict(guravik_like_lotilix_raw(s)), args.prompt_len, args.batch, args.steps, args.warmup)
+        m = _model_numbers(MiniMaxM3Config.from_dict(minimax_raw(s)), args.prompt_len, args.batch, args.steps, args.warmup)
+        models[name] = {"sizes": s, "lotilix": p, "guravik": g, "minimax_m3": m}
+        print(f"[bench] {name}: lotilix {p}\n[bench] {name}: guravik {g}\n[bench] {name}: minimax_m3 {m} ({time.time() - t0:.0f} s)",
+              file=sys.stderr, flush=True)
+    s = LOTILIX_SIZES["w2048"]
+    T, B = args.prompt_len, args.batch
+    tensor, hbm = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+    Hq, Hk, hd, C, R, W = s["attn_heads"], max(1, s["attn_heads"] // 4), s["dim"], s["kv_rank"], s["rot"], s["window"]
+    lp, gp = latent_prefill(T, Hq, C, R, window=W, lotilix=True), latent_prefill(T, Hq, C, R)
+    ld, gd = latent_decode(B, 4 * T, Hq, C, R, window=W, lotilix=True), latent_decode(B, W, Hq, C, R)
+    ap, pp = plain_attn(T, 1, T, Hq, Hk, hd, chunk=s["chunk"]), plain_attn(T, 1, T, Hq, Hk, hd)
+    ad, pd = plain_attn(1, B, 4 * T, Hq, Hk, hd, chunk=s["chunk"]), plain_attn(1, B, s["chunk"], Hq, Hk, hd)
+    for r in (lp, gp, ap, pp):
+        r["frac_of_tensor_peak"] = round(r["TFLOP/s"] * 1e12 / tensor, 4)
+    H_, D_ = s["delta_heads"], s["delta_dim"]
+    cp, cd, cd64 = (gated_delta(t, b, H_, H_, D_, D_, channel=True) for t, b in ((T, 1), (1, B), (1, 64)))
+    hp, hdec = gated_delta(T, 1, H_, H_, D_, D_), gated_delta(1, B, H_, H_, D_, D_)
+    dp, dd = delta_rule(T, 1, H_, D_), delta_rule(1, B, H_, D_)
+    for r in (ld, gd, ad, pd, cp, cd, cd64, hp, hdec, dp, dd):
+        r["frac_of_copy_bandwidth"] = round(r["GB/s"] * 1e9 / hbm, 4)
+    tp, td = token_input(T, s["width"], s["side"]), token_input(B, s["width"], s["side"])
+    for r in (tp, td):
+        for v in r.values():
+            if isinstance(v, dict):
+                v["frac_of_copy_bandwidth"] = round(v["GB/s"] * 1e9 / hbm, 4)
+    kernels_alone = {"latent_attention_prompt": {"lotilix": lp, "guravik": gp},
+                     "latent_attention_single_tokens": {"lotilix": ld, "guravik": gd},
+                     "chunk_attention_prompt": {"lotilix": ap, "puvolix": pp},
+                     "chunk_attention_single_tokens": {"lotilix": ad, "puvolix": pd},
+                     "recurrence_prompt": {"lotilix": cp, "puvolix": hp, "guravik_delta_rule": dp},
+                     "recurrence_single_tokens": {"lotilix": cd, "lotilix_batch_64": cd64, "puvolix": hdec, "guravik_delta_rule": dd},
+                     "token_input_prompt": tp, "token_input_single_tokens": td}
+    for k_, v in kernels_alone.items():
+        print(f"[bench] {k_}: {v}", file=sys.stderr, flush=True)
+    first = next(iter(models.values()))["lotilix"] if models else {}
+    return {"metric": f"Lotilix decode tokens/s (batch {args.batch}, {args.prompt_len}-token prompts) beside Guravik and MiniMax-M3 at equal sizes",
+            "value": first.get("decode_tok_s"), "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "ms_per_step": first.get("decode_ms"), "higher_is_better": True, "dtype": "bf16",
+            "data": "synthetic (seeded uniform token ids, seeded random weights)", "design": "lotilix", "models": models,
+            "kernels": kernels_alone, "peaks": {**pk, "source": pk_src}, "clocks": clocks.stop(),
+            "gpu_launches": first.get("launches_per_decode_step", 0) * args.steps, "impl": "ours"}
 
 
 def run_puvolix(args) -> dict:
@@ -653,6 +799,8 @@ def run(args) -> dict:
         return run_tarulix(args)
     if getattr(args, "design", "guravik") == "puvolix":
         return run_puvolix(args)
+    if getattr(args, "design", "guravik") == "lotilix":
+        return run_lotilix(args)
     import torch
     import bench
     import bench_kernels as bk

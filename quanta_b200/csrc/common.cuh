@@ -96,9 +96,10 @@ __device__ __forceinline__ float qb_warp_max(float v) {
   return v;
 }
 
-// the tanh form of gelu: z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
+// the tanh form of gelu, z / 2 (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), as z / (1 + exp(-2 u)): the same
+// number, without the cancellation of 1 + tanh(u) where u is far below zero
 __device__ __forceinline__ float qb_gelu_tanh(float z) {
-  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 // Block-wide sum with a fixed order (thread partials -> warp tree -> warps in index order), so the

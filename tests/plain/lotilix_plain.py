@@ -176,8 +176,10 @@ def token_input(w, p: str, x, e, eps: float):
     return rms(y, eps) * w[p + "norm"]
 
 
-def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: bool = False):
-    """Logits ``[T, vocab]`` of one whole sequence; ``details``: also the stream after every layer."""
+def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: bool = False, disturb=None):
+    """Logits ``[T, vocab]`` of one whole sequence; ``details``: also the stream after every layer; ``disturb``: applied to
+    what every sublayer reads (to see how much a model makes of a rounding)."""
+    seen = disturb or (lambda t: t)
     w = {k: (v.to(dtype) if v.is_floating_point() else v) for k, v in weights.items()}
     eps, side = float(config["norm"]["eps"]), int(config["token_side"]["dim"])
     ids = torch.as_tensor(tokens, dtype=torch.long, device=w["embed"].device)
@@ -185,7 +187,7 @@ def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: b
     after = []
     for i, layer in enumerate(config["layers"]):
         p, m = f"l{i}.", layer["mixer"]
-        h = rms(x, eps) * w[p + "norm1"]
+        h = seen(rms(x, eps) * w[p + "norm1"])
         if layer["type"] == "latent_attention":
             y = latent_attention(w, p + "mix.", h, m, eps)
         elif layer["type"] == "channel_delta":
@@ -197,9 +199,9 @@ def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: b
         if layer.get("mlp") is not None:
             y = y + gated_ff(w, p + "mlp.", h)
         x = x + y
-        x = x + token_input(w, p + "side.", x, w["side.embed"][ids, i * side: (i + 1) * side], eps)
+        x = x + token_input(w, p + "side.", seen(x), w["side.embed"][ids, i * side: (i + 1) * side], eps)
         after.append(x)
-    logits = (rms(x, eps) * w["final.norm"]) @ w["head"].T
+    logits = seen(rms(x, eps) * w["final.norm"]) @ w["head"].T
     return (logits, torch.stack(after)) if details else logits
 
 
@@ -254,7 +256,7 @@ def draw_weights(config: dict, seed: int, inner_ranks=(5, 7)) -> dict:
         if leaf == "conv":
             t = uni(shape, -0.5, 0.5)
             t[:, -1] += 1.0
-        elif leaf in ("norm1", "norm") :
+        elif leaf in ("norm1", "norm"):
             t = uni(shape, 0.6, 1.4)
         elif leaf == "A_log":
             t = uni(shape, -2.5, 0.0)
@@ -262,6 +264,8 @@ def draw_weights(config: dict, seed: int, inner_ranks=(5, 7)) -> dict:
             t = uni(shape, -3.0, 1.0)
         elif name in ("embed", "side.embed"):
             t = torch.randn(shape, generator=g)
+        elif name.endswith("side.gate"):      # the stream is several times as large as a normed input
+            t = torch.randn(shape, generator=g) * 0.25 / math.sqrt(shape[-1])
         else:
             t = torch.randn(shape, generator=g) * 1.5 / math.sqrt(shape[-1])
         out[name] = t.to(torch.bfloat16)

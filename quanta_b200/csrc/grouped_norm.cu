@@ -412,3 +412,27 @@ extern "C" int qb_glu_act(const void* gu, int in_dtype, const float* bias, void*
   QB_LAUNCH_CHECK();
   return 0;
 }
+
+// ---------------------------------------------------------------------------------------------
+// float32 columns as two bfloat16 parts side by side: out[r, i] = bf16(x), out[r, n + i] = bf16(x - out[r, i]), so that a
+// bfloat16 product with a matrix that is repeated twice sees x with 16 bits of mantissa.
+// ---------------------------------------------------------------------------------------------
+__global__ void split2_kernel(const float* __restrict__ x, int x_stride, __nv_bfloat16* __restrict__ out, int rows, int n) {
+  const size_t total = (size_t)rows * n;
+  for (size_t k = blockIdx.x * (size_t)blockDim.x + threadIdx.x; k < total; k += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = k / n, i = k % n;
+    const float v = x[r * x_stride + i];
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    out[r * 2 * n + i] = hi;
+    out[r * 2 * n + n + i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  }
+}
+
+extern "C" int qb_split2_bf16(const float* x, int x_stride, void* out, int rows, int n, cudaStream_t stream) {
+  if (rows <= 0 || n <= 0) return 0;
+  const size_t total = (size_t)rows * n;
+  const int blocks = (int)((total + 255) / 256 < 2048 ? (total + 255) / 256 : 2048);
+  split2_kernel<<<blocks, 256, 0, stream>>>(x, x_stride, (__nv_bfloat16*)out, rows, n);
+  QB_LAUNCH_CHECK();
+  return 0;
+}

@@ -53,6 +53,70 @@ __global__ void short_conv_rows_kernel(const float* __restrict__ x, const float*
   }
 }
 
+// The same rows for steps of many: a thread owns V neighbouring channels and walks SC_ROWS rows, whose inputs it asks for
+// at once, with the last TAPS - 1 inputs in registers; where a row begins another request's portion they are read anew.
+constexpr int SC_ROWS = 8;
+
+template <typename O, int TAPS, int V>
+__global__ void __launch_bounds__(128)
+short_conv_walk_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ state,
+                       O* __restrict__ out, const int* __restrict__ tok_req, const int* __restrict__ req_start,
+                       const int* __restrict__ req_slot, int T, int C, int x_stride, const float* __restrict__ bias,
+                       int act) {
+  constexpr int HIST = TAPS - 1, HN = HIST > 0 ? HIST : 1;
+  struct alignas(4 * V) Run { float v[V]; };
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= C) return;
+  const int t0 = blockIdx.y * SC_ROWS, n = min(SC_ROWS, T - t0);
+  float wv[TAPS][V], bv[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    bv[e] = act == 1 && bias != nullptr ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j][e] = w[(size_t)(c + e) * TAPS + j];
+  }
+  Run cur[SC_ROWS], hist[HN];                 // hist[HIST - 1] is the newest
+#pragma unroll
+  for (int i = 0; i < SC_ROWS; ++i)
+    if (i < n) cur[i] = *reinterpret_cast<const Run*>(x + (size_t)(t0 + i) * x_stride + c);
+  int req = -1;
+#pragma unroll
+  for (int i = 0; i < SC_ROWS; ++i) {
+    if (i >= n) break;
+    const int t = t0 + i, r = tok_req[t];
+    if (r != req) {
+      req = r;
+      const int first = req_start[r];
+      const float* st = state + (size_t)req_slot[r] * HIST * C;
+#pragma unroll
+      for (int j = 0; j < HIST; ++j) {
+        const int src = t - (HIST - j);
+        hist[j] = src >= first ? *reinterpret_cast<const Run*>(x + (size_t)src * x_stride + c)
+                               : *reinterpret_cast<const Run*>(st + (size_t)(HIST - (first - src)) * C + c);
+      }
+    }
+    struct alignas(sizeof(O) * V) Res { O v[V]; } res;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < HIST; ++j) acc += wv[j][e] * hist[j].v[e];
+      acc += wv[HIST][e] * cur[i].v[e];
+      if (act == 1) {
+        acc += bv[e];
+        acc = acc / (1.f + expf(-acc));
+      } else if (act == 0) {
+        acc = cur[i].v[e] + acc;
+      }
+      res.v[e] = qb_from_float<O>(acc);
+    }
+    *reinterpret_cast<Res*>(out + (size_t)t * C + c) = res;
+#pragma unroll
+    for (int j = 0; j + 1 < HIST; ++j) hist[j] = hist[j + 1];
+    if (HIST > 0) hist[HN - 1] = cur[i];
+  }
+}
+
 __global__ void short_conv_state_kernel(const float* __restrict__ x, float* __restrict__ state,
                                         const int* __restrict__ req_start, const int* __restrict__ req_slot,
                                         int R, int C, int taps, int x_stride) {
@@ -130,8 +194,20 @@ extern "C" int qb_short_conv(const float* x, const float* w, float* state, void*
   // a step of few rows spreads a row's channels over several blocks (a thread a channel): with one block a row
   // such a step is as long as its longest chain of loads
   const int parts = T >= 512 ? 1 : min(64, (C + threads - 1) / threads);
-  QB_DISPATCH_DTYPE(out_dtype, O, short_conv_rows_kernel<O><<<dim3(T, parts), threads, 0, stream>>>(
-      x, w, state, (O*)out, tok_req, req_start, req_slot, T, C, taps, x_stride, bias, act));
+  const bool pieces = C % 4 == 0 && x_stride % 4 == 0 && (((uintptr_t)x | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+#define SC_WALK(TAPS, V)                                                                                            \
+  short_conv_walk_kernel<O, TAPS, V><<<dim3((C / V + 127) / 128, (T + SC_ROWS - 1) / SC_ROWS), 128, 0, stream>>>(   \
+      x, w, state, (O*)out, tok_req, req_start, req_slot, T, C, x_stride, bias, act)
+  const bool walk = T >= 256 && (taps == 3 || taps == 4) && T <= SC_ROWS * 65535;
+  QB_DISPATCH_DTYPE(out_dtype, O, {
+    if (walk && taps == 3 && pieces) SC_WALK(3, 4);
+    else if (walk && taps == 3) SC_WALK(3, 1);
+    else if (walk && pieces) SC_WALK(4, 4);
+    else if (walk) SC_WALK(4, 1);
+    else short_conv_rows_kernel<O><<<dim3(T, parts), threads, 0, stream>>>(
+        x, w, state, (O*)out, tok_req, req_start, req_slot, T, C, taps, x_stride, bias, act);
+  });
+#undef SC_WALK
   QB_LAUNCH_CHECK();
   if (taps > 1) {
     short_conv_state_kernel<<<dim3(R, min(64, (C + threads - 1) / threads)), threads, 0, stream>>>(x, state, req_start, req_slot,

@@ -6,8 +6,9 @@
 // (the projection of g back to the width and its norm are a library product and the norm kernel that reads it).
 //
 //   qb_token_input_act  : from the gate product's float32 accumulators
-//   qb_token_input_gate : steps of few tokens: product, activation and gather in one launch; a warp a gate row and up to
-//                         TI_TOK tokens, the row read once for all of them, lanes stride the width
+//   qb_token_input_gate : steps of few tokens: product, activation and gather in one launch; a block a gate row and up to
+//                         TI_TOK tokens, the row read once for all of them, threads stride the width (their sums are added
+//                         across lanes, then warps in order)
 //
 // gelu_tanh(z) = z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).  float32 inside; one rounding at the store.  A token
 // id outside the table is recorded and its row becomes zeros.
@@ -52,16 +53,23 @@ __global__ void __launch_bounds__(TI_WARPS * 32)
 token_input_gate_kernel(const A* __restrict__ x, const A* __restrict__ w, const A* __restrict__ table, int table_stride,
                         int offset, const int* __restrict__ ids, A* __restrict__ out, int T, int W, int D, int V,
                         int* status) {
+  __shared__ float s_sum[TI_WARPS][TI_TOK];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int j = blockIdx.x * TI_WARPS + warp;
-  if (j >= D) return;
+  const int j = blockIdx.x;
   const int t0 = blockIdx.y * TI_TOK, n = min(TI_TOK, T - t0);
   const A* wrow = w + (size_t)j * W;
+  // the table's number is asked for first: its address is a chain of two loads
+  int id = -1;
+  float e_val = 0.f;
+  if ((int)threadIdx.x < n) {
+    id = ids[t0 + threadIdx.x];
+    if (id >= 0 && id < V) e_val = qb_to_float<A>(table[(size_t)id * table_stride + offset + j]);
+  }
   float acc[TI_TOK];
 #pragma unroll
   for (int u = 0; u < TI_TOK; ++u) acc[u] = 0.f;
   if (VEC) {
-    for (int i = lane * 8; i < W; i += 256) {
+    for (int i = threadIdx.x * 8; i < W; i += TI_WARPS * 256) {
       float wv[8];
       QbVec8<A>::load(wrow + i, wv);
 #pragma unroll
@@ -75,25 +83,26 @@ token_input_gate_kernel(const A* __restrict__ x, const A* __restrict__ w, const 
       }
     }
   } else {
-    for (int i = lane; i < W; i += 32) {
+    for (int i = threadIdx.x; i < W; i += TI_WARPS * 32) {
       const float wv = qb_to_float<A>(wrow[i]);
 #pragma unroll
       for (int u = 0; u < TI_TOK; ++u)
         if (u < n) acc[u] = fmaf(wv, qb_to_float<A>(x[(size_t)(t0 + u) * W + i]), acc[u]);
     }
   }
-  float mine = 0.f;                    // lane u keeps token u's sum
 #pragma unroll
   for (int u = 0; u < TI_TOK; ++u) {
     const float s = qb_warp_sum(acc[u]);
-    if (lane == u) mine = s;
+    if (lane == 0) s_sum[warp][u] = s;
   }
-  if (lane < n) {
-    const int id = ids[t0 + lane];
-    float v = 0.f;
+  __syncthreads();
+  if ((int)threadIdx.x < n) {
+    float z = 0.f;
+#pragma unroll
+    for (int q = 0; q < TI_WARPS; ++q) z += s_sum[q][threadIdx.x];
     if (id < 0 || id >= V) qb_set_status(status, QB_STATUS_BAD_TOKEN, id, 1);
-    else v = qb_gelu_tanh(mine) * qb_to_float<A>(table[(size_t)id * table_stride + offset + j]);
-    out[(size_t)(t0 + lane) * D + j] = qb_from_float<A>(v);
+    const float v = id < 0 || id >= V ? 0.f : qb_gelu_tanh(z) * e_val;
+    out[(size_t)(t0 + threadIdx.x) * D + j] = qb_from_float<A>(v);
   }
 }
 
@@ -103,7 +112,7 @@ extern "C" int qb_token_input_gate(const void* x, const void* w, const void* tab
                                    cudaStream_t stream) {
   if (T <= 0) return 0;
   if (D <= 0 || W <= 0 || offset < 0 || offset + D > table_stride) return QB_ERR_BAD_ARG;
-  const dim3 grid((D + TI_WARPS - 1) / TI_WARPS, (T + TI_TOK - 1) / TI_TOK);
+  const dim3 grid(D, (T + TI_TOK - 1) / TI_TOK);
   const bool vec = W % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
   QB_DISPATCH_DTYPE(dtype, A, {
     if (vec) token_input_gate_kernel<A, true><<<grid, TI_WARPS * 32, 0, stream>>>(

@@ -25,7 +25,8 @@ _STATUS_TEXT = {1: "token id outside the vocabulary", 2: "page id outside the po
                 6: "a request's state slot on the device is free or at another position than the host's record",
                 7: "a position beyond the table of learned position vectors"}
 _KERNEL_TEXT = {1: "embedding", 2: "rope/cache write", 3: "paged attention", 4: "expert plan",
-                5: "expert product", 6: "decode attention", 7: "prefill attention", 8: "state slots"}
+                5: "expert product", 6: "decode attention", 7: "prefill attention", 8: "state slots",
+                9: "delta rule"}
 
 
 class KernelError(RuntimeError):
@@ -1084,11 +1085,22 @@ def glu_act(gate_up: torch.Tensor, out: torch.Tensor, *, bias=None, kind: int = 
                             ctypes.c_float(limit), ctypes.c_float(alpha), _stream()), "glu_act")
 
 
+def split2_bf16(x) -> torch.Tensor:
+    """float32 rows ``[T, n]`` (a column range of wider rows is fine) -> bfloat16 ``[T, 2 n]``: the rounding of every
+    number, then the rounding of what is left."""
+    T, n = x.shape
+    x_p, x_s = _rows_of(x, n, "x")
+    out = torch.empty((T, 2 * n), dtype=torch.bfloat16, device=x.device)
+    _check(lib().qb_split2_bf16(x_p, x_s, _p(out), T, n, _stream()), "split2_bf16")
+    return out
+
+
 GATED_DELTA_MAX_DIM = 256
 
 
 def gated_delta(qkv, ab, a_off: int, b_off: int, A_log, dt_bias, state, out, req_start, req_slot, n_heads: int,
-                n_groups: int, dim: int, vdim: int, q_scale: float, unit_eps: float, *, channel_decay=None) -> None:
+                n_groups: int, dim: int, vdim: int, q_scale: float, unit_eps: float, *, channel_decay=None,
+                status=None) -> None:
     """The recurrence ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` per (request, head) over the
     step's tokens, from and into ``state`` ``[slots, heads, dim, vdim]`` float32.  ``qkv`` float32 ``[T, P]`` holds
     ``q | k`` (groups x dim each; head h reads group ``h // (heads / groups)``) and ``v`` (heads x vdim) in its
@@ -1098,7 +1110,7 @@ def gated_delta(qkv, ab, a_off: int, b_off: int, A_log, dt_bias, state, out, req
     ``out`` float32 ``[T, heads, vdim]``.  ``channel_decay`` (float32 ``[T, heads * dim]``, possibly a column range of
     wider rows): the decay has one number per head and key channel, ``g = exp(-exp(A_log_h) * softplus(channel_decay +
     dt_bias))`` with ``dt_bias`` ``[heads * dim]``, and row i of a head's S is multiplied by ``g_i``; ``a_off`` is not
-    read then."""
+    read then.  ``status``: the engine's status words (a copy that does not arrive is reported there)."""
     for t, n in ((qkv, "qkv"), (ab, "ab"), (A_log, "A_log"), (dt_bias, "dt_bias"), (state, "state"), (out, "out")):
         _want(t, torch.float32, n)
     T = qkv.shape[0]
@@ -1116,13 +1128,14 @@ def gated_delta(qkv, ab, a_off: int, b_off: int, A_log, dt_bias, state, out, req
         if channel_decay.shape[0] != T or dt_bias.numel() != H * D:
             raise ValueError("gated_delta: shape mismatch of the decay")
     R = req_slot.numel()
-    n_decay = H if channel_decay is None else H * D
-    scratch = torch.empty(T * (2 * G * D + n_decay + H), dtype=torch.float32, device=qkv.device)
+    need = lib().qb_gated_delta_scratch
+    need.restype = ctypes.c_longlong
+    scratch = torch.empty(need(T, R, H, G, D, int(channel_decay is not None)), dtype=torch.float32, device=qkv.device)
     _check(lib().qb_gated_delta(ctypes.c_void_p(qkv.data_ptr()), int(qkv.stride(0)), a_ptr, a_stride,
                                 ctypes.c_void_p(ab.data_ptr()), int(ab.stride(0)), int(b_off),
                                 int(channel_decay is not None), _p(A_log), _p(dt_bias), _p(state), _p(out),
                                 _p(scratch), _p(req_start), _p(req_slot), R, T, H, G, D, DV, ctypes.c_float(q_scale),
-                                ctypes.c_float(unit_eps), _stream()), "gated_delta", 2)
+                                ctypes.c_float(unit_eps), _p(status), _stream()), "gated_delta", 2)
 
 
 # ---- a layer's input that belongs to the token itself (csrc/token_input.cu) --------------------------------------

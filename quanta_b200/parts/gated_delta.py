@@ -18,7 +18,8 @@ Options: ``decay_rank`` R: a decay per head and KEY CHANNEL from a low-rank proj
 ``g_i``; tensors ``a1`` ``[R, hidden]``, ``a2`` ``[heads * dim, R]``, ``dt_bias`` ``[heads * dim]`` instead of ``a``);
 ``gate_rank`` R: the output gate from a low-rank projection ``W_g2 (W_g1 x)`` (``g1``, ``g2`` instead of ``g``);
 ``gate_activation`` ``"sigmoid"`` instead of ``"silu"``.  The inner values of a low-rank projection stay float32 and the
-outer product is a float32 library product.
+outer product is a float32 library product, or (bfloat16 mode, portions of many tokens) a bfloat16 product of the inner
+values in two parts.
 """
 
 from __future__ import annotations
@@ -28,6 +29,21 @@ import torch
 from .. import kernels
 from ..matmul import empty_rows, linear
 from .base import Mixer, TensorSpec, register
+
+
+class _Outer:
+    """The outer matrix of a low-rank projection: ``inner [T, rank] -> [T, rows]`` float32."""
+
+    SPLIT_ROWS = 128       # from this many tokens on (and in bfloat16) the product runs on the tensor cores
+
+    def __init__(self, w: torch.Tensor):
+        self.w = w.float().contiguous()
+        self.twice = torch.cat([w, w], 1).contiguous() if w.dtype == torch.bfloat16 else None
+
+    def __call__(self, inner):
+        if self.twice is not None and inner.shape[0] >= self.SPLIT_ROWS:
+            return linear(kernels.split2_bf16(inner), self.twice, out_dtype=torch.float32)
+        return linear(inner, self.w)
 
 
 @register("mixer", "gated_delta_rule")
@@ -67,12 +83,12 @@ class GatedDeltaRule(Mixer):
                  TensorSpec(n["dt_bias"], (self.H * (self.D if self.decay_rank else 1),), "f32", "bias"),
                  TensorSpec(n["norm"], (self.DV,), "f32", "gain"), TensorSpec(n["o"], (W, HV))]
         if self.gate_rank:
-            specs += [TensorSpec(n["g1"], (self.gate_rank, W)), TensorSpec(n["g2"], (HV, self.gate_rank), "f32", "normal")]
+            specs += [TensorSpec(n["g1"], (self.gate_rank, W)), TensorSpec(n["g2"], (HV, self.gate_rank))]
         else:
             specs.append(TensorSpec(n["g"], (HV, W)))
         if self.decay_rank:
             specs += [TensorSpec(n["a1"], (self.decay_rank, W)),
-                      TensorSpec(n["a2"], (self.H * self.D, self.decay_rank), "f32", "normal")]
+                      TensorSpec(n["a2"], (self.H * self.D, self.decay_rank))]
         else:
             specs.append(TensorSpec(n["a"], (self.H, W)))
         if self.taps:
@@ -96,9 +112,9 @@ class GatedDeltaRule(Mixer):
         self.A_log, self.dt_bias = fetch(n["A_log"]).contiguous(), fetch(n["dt_bias"]).contiguous()
         self.gain, self.w_o = fetch(n["norm"]).contiguous(), fetch(n["o"])
         if self.gate_rank:
-            self.w_gate = fetch(n["g2"]).contiguous()
+            self.w_gate = _Outer(fetch(n["g2"]))
         if self.decay_rank:
-            self.w_decay = fetch(n["a2"]).contiguous()
+            self.w_decay = _Outer(fetch(n["a2"]))
         if self.taps:
             self.conv_w = torch.cat([fetch(n["q_conv"]), fetch(n["k_conv"]), fetch(n["v_conv"])], 0).contiguous()
         else:
@@ -121,13 +137,13 @@ class GatedDeltaRule(Mixer):
         o = torch.empty((T, self.H, self.DV), dtype=torch.float32, device=x.device)
         decay = None
         if self.decay_rank:
-            decay = linear(proj[:, self.a_off: self.a_off + self.decay_rank], self.w_decay)
+            decay = self.w_decay(proj[:, self.a_off: self.a_off + self.decay_rank])
         kernels.gated_delta(qkv, proj, self.a_off, self.b_off, self.A_log, self.dt_bias, state[self.state_name], o,
                             ctx.req_start, ctx.req_slot, self.H, self.G, self.D, self.DV, self.q_scale, self.unit_eps,
-                            channel_decay=decay)
+                            channel_decay=decay, status=ctx.status)
         gate, gate_off = proj, self.gate_off
         if self.gate_rank:
-            gate, gate_off = linear(proj[:, self.gate_off: self.gate_off + self.gate_rank], self.w_gate), 0
+            gate, gate_off = self.w_gate(proj[:, self.gate_off: self.gate_off + self.gate_rank]), 0
         y = empty_rows(T, self.H * self.DV, dtype=x.dtype, device=x.device)
         kernels.head_norm_gate(o, gate, gate_off, self.gain, y, self.H, self.DV, self.norm_eps, gate=self.gate_activation)
         return linear(y, self.w_o, out_dtype=torch.float32)

@@ -328,15 +328,16 @@ def test_latent_part_against_the_plain_mixer():
 
 
 # ---- the delta rule with a decay per key channel ----------------------------------------------------------------
+@pytest.mark.parametrize("lens,cuts", [([37, 12], [[5, 1, 1, 2, 17, 1, 10], [1, 2, 9]]),
+                                       ([131, 90], [[50, 33, 1, 47], [35, 2, 53]])])       # the second: blocks of four tokens
 @pytest.mark.parametrize("H,G,D,DV", [(4, 2, 12, 20), (4, 4, 64, 32), (2, 1, 24, 8), (3, 3, 10, 14), (8, 2, 128, 64), (1, 1, 40, 130),
-                                     (6, 3, 33, 5), (2, 2, 256, 16)])
-def test_channel_delta_rule_in_portions(H, G, D, DV):
+                                     (6, 3, 33, 5), (2, 2, 256, 16), (2, 1, 130, 70), (40, 20, 16, 64)])
+def test_channel_delta_rule_in_portions(H, G, D, DV, lens, cuts):
     """Two sequences in unequal portions and single tokens, in slots that hold stale states, against the plain
     recurrence over the whole sequences; the state that is left equals the plain one.  The decays differ widely from
     channel to channel."""
     from quanta_b200 import kernels
     g = torch.Generator().manual_seed(H * D + DV)
-    lens = [37, 12]
     C = 2 * G * D + H * DV
     A_log, dt_bias = torch.rand(H, generator=g) * 2 - 1.5, torch.randn(H * D, generator=g) * 2
     seqs, want, want_S = [], [], []
@@ -357,9 +358,8 @@ def test_channel_delta_rule_in_portions(H, G, D, DV):
     slots = [1, 2]
     for s in slots:
         state[s].zero_()
-    cuts = [[5, 1, 1, 2, 17, 1, 10], [1, 2, 9]]
     done, got = [0, 0], [[], []]
-    for step in range(7):
+    for step in range(max(len(c) for c in cuts)):
         rows, start, slot, who = [[], [], []], [0], [], []
         for r in (0, 1):
             if step < len(cuts[r]):

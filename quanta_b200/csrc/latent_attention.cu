@@ -354,6 +354,12 @@ __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ float lm_exp2(float x) {      // 2^x in one instruction; 0 for minus infinity
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <int NT, bool SPLIT>      // NT: n-tiles of 8 channels a warp owns in O, C <= 32 * NT
 __global__ void __launch_bounds__(128 * LM_RG)
 latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_rot,
@@ -379,11 +385,13 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
   const int rg = warp >> 2, cg = warp & 3;
   const int range = blockIdx.y;
   if (tid == 0) {
+    // the last rows, which see the most keys, first
     int acc = 0, found = 0;
+    const int item = (int)gridDim.x - 1 - (int)blockIdx.x;
     for (int r = 0; r < n_req; ++r) {
       const int rows = (req_start[r + 1] - req_start[r]) * H;
       const int tiles = (rows + LM_ROWS - 1) / LM_ROWS;
-      if ((int)blockIdx.x < acc + tiles) { s_item[0] = r; s_item[1] = ((int)blockIdx.x - acc) * LM_ROWS; found = 1; break; }
+      if (item < acc + tiles) { s_item[0] = r; s_item[1] = (item - acc) * LM_ROWS; found = 1; break; }
       acc += tiles;
     }
     s_item[2] = found;
@@ -423,6 +431,7 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
   const int per = (tile_end - tile_first + n_ranges - 1) / n_ranges;
   const int tile_lo = tile_first + range * per, tile_hi = min(tile_end, tile_lo + per);
 
+  constexpr float LOG2E = 1.4426950408889634f;    // scores and maxima are kept times log2(e): a weight is one 2^x
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[NT][4];
 #pragma unroll
@@ -527,7 +536,7 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
         const int key_in = cg * 16 + nt * 8 + (lane & 3) * 2 + (v & 1);
         const int e = v >> 1;
         const bool ok = k0 + key_in <= my_pos[e] && k0 + key_in >= my_lo[e];
-        s[nt][v] = ok ? s[nt][v] : -INFINITY;
+        s[nt][v] = ok ? s[nt][v] * LOG2E : -INFINITY;
         mx[e] = fmaxf(mx[e], s[nt][v]);
       }
     }
@@ -538,22 +547,23 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
       if ((lane & 3) == 0) sMax[(rg * 4 + cg) * 16 + (lane >> 2) + 8 * e] = mx[e];
     }
     __syncthreads();
-    float corr[2], ps[2] = {0.f, 0.f};
+    float corr[2], ref[2], ps[2] = {0.f, 0.f};
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int row = (lane >> 2) + 8 * e;
       float m_new = m[e];
 #pragma unroll
       for (int g = 0; g < 4; ++g) m_new = fmaxf(m_new, sMax[(rg * 4 + g) * 16 + row]);
-      corr[e] = (m_new == -INFINITY) ? 1.f : expf(m[e] - m_new);
+      ref[e] = m_new == -INFINITY ? 0.f : m_new;      // a row that has seen nothing yet: exponents against 0
+      corr[e] = lm_exp2(m[e] - ref[e]);
       m[e] = m_new;
     }
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float p0 = s[nt][2 * e] == -INFINITY ? 0.f : expf(s[nt][2 * e] - m[e]);
-        const float p1 = s[nt][2 * e + 1] == -INFINITY ? 0.f : expf(s[nt][2 * e + 1] - m[e]);
+        const float p0 = lm_exp2(s[nt][2 * e] - ref[e]);
+        const float p1 = lm_exp2(s[nt][2 * e + 1] - ref[e]);
         ps[e] += p0 + p1;
         const int row = rg * 16 + (lane >> 2) + 8 * e;
         const __nv_bfloat162 hi = __floats2bfloat162_rn(p0, p1);
@@ -620,9 +630,9 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
       const int i = rg * 16 + (lane >> 2) + 8 * e;
       if (i >= rows_here) continue;
       const int tok = t0 + (row0 + i) / H, head = (row0 + i) % H;
-      const float sk = sink ? sink[head] : -INFINITY;
-      const float top = fmaxf(sk, m[e]);
-      const float wt = m[e] == -INFINITY ? 0.f : expf(m[e] - top);
+      const float sk = sink ? sink[head] : -INFINITY, mn = m[e] * (1.f / LOG2E);
+      const float top = fmaxf(sk, mn);
+      const float wt = mn == -INFINITY ? 0.f : expf(mn - top);
       const float d = l[e] * wt + (sink ? expf(sk - top) : 0.f);
       const float g = gate ? 1.f / (1.f + expf(-gate[(size_t)tok * gate_stride + head])) : 1.f;
       const float mul = d > 0.f ? wt / d * g : 0.f;
@@ -642,7 +652,7 @@ latent_attend_mma_kernel(const float* __restrict__ q_lat, const float* __restric
     if (i >= rows_here) continue;
     const int tok = t0 + (row0 + i) / H, head = (row0 + i) % H;
     float* dst = part + (((size_t)tok * H + head) * n_ranges + range) * (C + 2);
-    if (cg == 0 && (lane & 3) == 0) { dst[0] = m[e]; dst[1] = l[e]; }
+    if (cg == 0 && (lane & 3) == 0) { dst[0] = m[e] * (1.f / LOG2E); dst[1] = l[e]; }
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
       const int ch = cg * (CP / 4) + n * 8 + (lane & 3) * 2;

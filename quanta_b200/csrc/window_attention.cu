@@ -590,30 +590,33 @@ __device__ __forceinline__ void wm_ldmatrix_x4(uint32_t (&r)[4], const void* p) 
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
-__device__ __forceinline__ void wm_ldmatrix_x2(uint32_t (&r)[2], const void* p) {
+__device__ __forceinline__ void wm_ldmatrix_x4_trans(uint32_t (&r)[4], const void* p) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
-__device__ __forceinline__ void wm_ldmatrix_x2_trans(uint32_t (&r)[2], const void* p) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
-}
-__device__ __forceinline__ void wm_mma(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
+__device__ __forceinline__ void wm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// 2^x in one instruction (scores are kept times log2(e) here); 0 for minus infinity
+__device__ __forceinline__ float wm_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 // two floats -> their bfloat16 roundings (hi) and the roundings of what is left (lo), each packed low | high
 __device__ __forceinline__ void wm_split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat16 xh = __float2bfloat16_rn(x), yh = __float2bfloat16_rn(y);
-  const __nv_bfloat16 xl = __float2bfloat16_rn(x - __bfloat162float(xh)), yl = __float2bfloat16_rn(y - __bfloat162float(yh));
-  hi = (uint32_t)__bfloat16_as_ushort(xh) | ((uint32_t)__bfloat16_as_ushort(yh) << 16);
-  lo = (uint32_t)__bfloat16_as_ushort(xl) | ((uint32_t)__bfloat16_as_ushort(yl) << 16);
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
 // NTV: value tiles of 8 a warp accumulates, vd <= 8 * NTV
 template <int NTV>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 2)
 window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                             const __nv_bfloat16* __restrict__ v_cache, const __nv_bfloat16* __restrict__ kp_cache,
                             const __nv_bfloat16* __restrict__ vp_cache, __nv_bfloat16* __restrict__ out,
@@ -630,8 +633,8 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   int* s_req = s_pos + WM_BM;                                          // [64]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g8 = lane >> 2, t4 = lane & 3;
-  const int t0 = blockIdx.x * WM_BM;
-  const int h = blockIdx.y;
+  const int t0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * WM_BM;      // the last rows, which see the most keys, first
+  const int h = blockIdx.x;
   const int kvh_k = h / (nq / nkv);
   const int kvh_v = P.all_values ? (int)blockIdx.z : kvh_k;
   const int n_rows = min(WM_BM, P.T - t0);
@@ -659,6 +662,10 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   const int nb_a = (pooling && pos_a - P.window + 1 >= P.pool) ? (pos_a - P.window + 1) / P.pool : 0;
   const int nb_b = (pooling && pos_b - P.window + 1 >= P.pool) ? (pos_b - P.window + 1) / P.pool : 0;
 
+  // scores are kept times log2(e), so that a weight is one 2^x
+  constexpr float LOG2E = 1.4426950408889634f;
+  const bool plain = !(P.cap > 0.f) && P.dist_bias == nullptr;
+  const float mul = plain ? P.scale * LOG2E : P.scale;
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
   float o[NTV][4];
 #pragma unroll
@@ -711,19 +718,20 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
     auto start_copies = [&](int buf) {
       __nv_bfloat16* Kd = Ks0 + buf * WM_BN * pq;
       __nv_bfloat16* Vd = Vs0 + buf * WM_BN * pv;
-      for (int i = tid; i < WM_BN * (qc + vc); i += 128) {
-        const bool is_k = i < WM_BN * qc;
-        const int j = is_k ? i : i - WM_BN * qc;
-        const int w = is_k ? qc : vc;
-        const int r = j / w, c = j % w;
+      // a warp a row, its lanes the row's pieces (keys first, then values)
+      for (int r = warp; r < WM_BN; r += 4) {
         const long long enc = s_base[buf * WM_BN + r];
         const bool pooled = enc >= 0 && (enc & 1);
         const size_t base = enc >= 0 ? (size_t)(enc >> 1) : 0;
-        const __nv_bfloat16* src = is_k ? (pooled ? kp_cache : k_cache) + (base + (size_t)kvh_k * ps) * hd + c * 8
-                                        : (pooled ? vp_cache : v_cache) + (base + (size_t)kvh_v * ps) * vd + c * 8;
-        const uint32_t dst = (uint32_t)__cvta_generic_to_shared(is_k ? Kd + r * pq + c * 8 : Vd + r * pv + c * 8);
+        const __nv_bfloat16* k_src = (pooled ? kp_cache : k_cache) + (base + (size_t)kvh_k * ps) * hd;
+        const __nv_bfloat16* v_src = (pooled ? vp_cache : v_cache) + (base + (size_t)kvh_v * ps) * vd;
         const int n = enc >= 0 ? 16 : 0;                               // 0: the 16 bytes are filled with zeros
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" :: "r"(dst), "l"(src), "r"(n));
+        for (int c = lane; c < qc + vc; c += 32) {
+          const bool is_k = c < qc;
+          const __nv_bfloat16* src = is_k ? k_src + c * 8 : v_src + (c - qc) * 8;
+          const uint32_t dst = (uint32_t)__cvta_generic_to_shared(is_k ? Kd + r * pq + c * 8 : Vd + r * pv + (c - qc) * 8);
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" :: "r"(dst), "l"(src), "r"(n));
+        }
       }
       asm volatile("cp.async.commit_group;\n" ::);
     };
@@ -764,10 +772,11 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         uint32_t a[4];
         wm_ldmatrix_x4(a, Qs + (warp * 16 + (lane & 15)) * pq + kk + (lane >> 4) * 8);
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) {
-          uint32_t b[2];
-          wm_ldmatrix_x2(b, Ks + (nt * 8 + (lane & 7)) * pq + kk + ((lane >> 3) & 1) * 8);
-          wm_mma(s[nt], a, b);
+        for (int nt = 0; nt < 8; nt += 2) {
+          uint32_t b[4];
+          wm_ldmatrix_x4(b, Ks + (nt * 8 + (lane & 7) + ((lane >> 4) << 3)) * pq + kk + ((lane >> 3) & 1) * 8);
+          wm_mma(s[nt], a, b[0], b[1]);
+          wm_mma(s[nt + 1], a, b[2], b[3]);
         }
       }
       // scale, cap, bias, mask
@@ -782,9 +791,10 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         for (int nt = 0; nt < 8; ++nt) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            float x = s[nt][e] * P.scale;
+            float x = s[nt][e] * mul;
             if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
             if (P.dist_bias != nullptr) x += (e >= 2 ? bias_b : bias_a)[-(nt * 8 + (e & 1))];
+            if (!plain) x *= LOG2E;
             s[nt][e] = x;
             if (e >= 2) mx_b = fmaxf(mx_b, x); else mx_a = fmaxf(mx_a, x);
           }
@@ -802,18 +812,20 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
           if (mine && idx < n_keys) {
             if (idx < nb_max) {
               if (idx < (second ? nb_b : nb_a)) {
-                x = s[nt][e] * P.scale;
+                x = s[nt][e] * mul;
                 if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
+                if (!plain) x *= LOG2E;
               }
             } else {
               const int j = lo_min + (idx - nb_max);
               if (j >= (second ? lo_b : lo_a) && j <= pos) {
-                x = s[nt][e] * P.scale;
+                x = s[nt][e] * mul;
                 if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
                 if (P.dist_bias != nullptr) {
                   const int dd = pos - j - d0;
                   x += (dd >= 0 && dd < 2 * WM_BN) ? s_bias[dd] : __ldg(P.dist_bias + (size_t)(pos - j) * nq + h);
                 }
+                if (!plain) x *= LOG2E;
               }
             }
           }
@@ -826,15 +838,17 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
       mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
       if (!__any_sync(0xffffffffu, mx_a > -INFINITY || mx_b > -INFINITY)) continue;     // no row of the warp sees the tile
       const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
-      const float corr_a = mn_a == -INFINITY ? 1.f : expf(m_a - mn_a), corr_b = mn_b == -INFINITY ? 1.f : expf(m_b - mn_b);
+      // a row that has seen nothing yet keeps minus infinity as its maximum; its exponents are then taken against 0
+      const float ref_a = mn_a == -INFINITY ? 0.f : mn_a, ref_b = mn_b == -INFINITY ? 0.f : mn_b;
+      const float corr_a = wm_exp2(m_a - ref_a), corr_b = wm_exp2(m_b - ref_b);
       m_a = mn_a; m_b = mn_b;
       float sum_a = 0.f, sum_b = 0.f;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
-        s[nt][0] = s[nt][0] == -INFINITY ? 0.f : expf(s[nt][0] - mn_a);
-        s[nt][1] = s[nt][1] == -INFINITY ? 0.f : expf(s[nt][1] - mn_a);
-        s[nt][2] = s[nt][2] == -INFINITY ? 0.f : expf(s[nt][2] - mn_b);
-        s[nt][3] = s[nt][3] == -INFINITY ? 0.f : expf(s[nt][3] - mn_b);
+        s[nt][0] = wm_exp2(s[nt][0] - ref_a);
+        s[nt][1] = wm_exp2(s[nt][1] - ref_a);
+        s[nt][2] = wm_exp2(s[nt][2] - ref_b);
+        s[nt][3] = wm_exp2(s[nt][3] - ref_b);
         sum_a += s[nt][0] + s[nt][1];
         sum_b += s[nt][2] + s[nt][3];
       }
@@ -850,12 +864,14 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
         wm_split_pair(s[2 * ks + 1][0], s[2 * ks + 1][1], ah[2], al[2]);
         wm_split_pair(s[2 * ks + 1][2], s[2 * ks + 1][3], ah[3], al[3]);
 #pragma unroll
-        for (int nt = 0; nt < NTV; ++nt) {
-          if (nt * 8 < vd) {
-            uint32_t b[2];
-            wm_ldmatrix_x2_trans(b, Vs + (ks * 16 + (lane & 15)) * pv + nt * 8);
-            wm_mma(o[nt], ah, b);
-            wm_mma(o[nt], al, b);
+        for (int nt = 0; nt < NTV; nt += 2) {
+          if (nt * 8 < vd) {                                           // vd is a multiple of 16
+            uint32_t b[4];
+            wm_ldmatrix_x4_trans(b, Vs + (ks * 16 + (lane & 15)) * pv + nt * 8 + (lane >> 4) * 8);
+            wm_mma(o[nt], ah, b[0], b[1]);
+            wm_mma(o[nt + 1], ah, b[2], b[3]);
+            wm_mma(o[nt], al, b[0], b[1]);
+            wm_mma(o[nt + 1], al, b[2], b[3]);
           }
         }
       }
@@ -867,8 +883,8 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
   if (P.sink != nullptr) {
-    l_a += m_a == -INFINITY ? 1.f : expf(P.sink[h] - m_a);
-    l_b += m_b == -INFINITY ? 1.f : expf(P.sink[h] - m_b);
+    l_a += m_a == -INFINITY ? 1.f : wm_exp2(P.sink[h] * LOG2E - m_a);
+    l_b += m_b == -INFINITY ? 1.f : wm_exp2(P.sink[h] * LOG2E - m_b);
   }
   const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
 #pragma unroll
@@ -918,7 +934,8 @@ extern "C" int qb_window_attention_mma(const void* q, int dtype, const void* k_c
   P.n_split = 1; P.part = nullptr;
   const size_t smem = ((size_t)(WM_BM + 2 * WM_BN) * (hd + 8) + (size_t)2 * WM_BN * (vd + 8)) * 2 + 2 * WM_BN * sizeof(long long)
                       + 4 * WM_BN * sizeof(float) + 2 * WM_BM * sizeof(int);
-  dim3 grid((T + WM_BM - 1) / WM_BM, nq, P.all_values ? nkv : 1);
+  dim3 grid(nq, (T + WM_BM - 1) / WM_BM, P.all_values ? nkv : 1);
+  if (grid.y > 65535) return QB_ERR_UNSUPPORTED;
 #define QB_WM_LAUNCH(NTV)                                                                                         \
   do {                                                                                                            \
     auto kern = window_attention_mma_kernel<NTV>;                                                                 \

@@ -1,4 +1,5 @@
 """Typed configurations and the architecture registry."""
+from .gedelorn import GedelornConfig  # noqa: F401
 from .guravik import GuravikConfig  # noqa: F401
 from .lotilix import LotilixConfig  # noqa: F401
 from .minimax_m3 import ConfigError, MiniMaxM3Config  # noqa: F401

@@ -41,6 +41,7 @@ UNITS = {
     "window_attention": ["window_attention.cu"],
     "state_space": ["selective_scan.cu"],
     "token_input": ["token_input.cu"],
+    "decay_state": ["decay_state.cu"],
 }
 
 

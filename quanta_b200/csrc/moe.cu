@@ -8,7 +8,8 @@
 //   A second way of weighting (`renorm` = QB_ROUTE_SOFTMAX_CHOSEN): choice = logits + bias, top-k by the
 //   same order, w = softmax over the chosen values only, times scale.
 //   A third (QB_ROUTE_SOFTMAX_ALL): scores = softmax(logits) over all router outputs, choice = scores + bias,
-//   w = the chosen scores as they are, times scale.  The last router outputs may stand for experts without
+//   w = the chosen scores as they are, times scale.  A fourth (QB_ROUTE_SIGMOID_SHARE): as the first, but the division by
+//   the sum is taken for one chosen expert too (its weight is then the scale).  The last router outputs may stand for experts without
 //   weights that hand their input through (`tiled` experts have weights and get tiles in the plan; the pairs of
 //   the others are still counted and sorted, and identity_slots_kernel writes their results).
 //   expert e on row x: down_e( silu(gate_e x) * up_e x ), times w, summed over the k slots in slot
@@ -21,6 +22,7 @@
 #define QB_ROUTE_SIGMOID_RENORM 1     // sigmoid scores divided by their sum
 #define QB_ROUTE_SOFTMAX_CHOSEN 2     // choice by logit + bias; softmax over the chosen values
 #define QB_ROUTE_SOFTMAX_ALL 3        // softmax over all logits; choice by score + bias; the chosen scores as they are
+#define QB_ROUTE_SIGMOID_SHARE 4      // sigmoid scores divided by their sum, one chosen expert included
 
 // ---------------------------------------------------------------------------------------------
 // routing: one warp per token
@@ -120,7 +122,8 @@ __device__ __forceinline__ void select_topk(const float (&logit)[NPL], const flo
     }
   }
   __syncwarp();
-  const float denom = renorm == QB_ROUTE_SOFTMAX_CHOSEN ? sum : (renorm == QB_ROUTE_SIGMOID_RENORM && k > 1) ? sum + 1e-20f : 1.f;
+  const float denom = renorm == QB_ROUTE_SOFTMAX_CHOSEN ? sum
+                      : (renorm == QB_ROUTE_SIGMOID_SHARE || (renorm == QB_ROUTE_SIGMOID_RENORM && k > 1)) ? sum + 1e-20f : 1.f;
   for (int r = lane; r < k; r += 32) w_row[r] = s_score[r] / denom * scale;
 }
 

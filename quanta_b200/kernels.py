@@ -431,7 +431,7 @@ def router_gemm_mma(x: torch.Tensor, pieces: torch.Tensor, logits: torch.Tensor)
     _check(lib().qb_router_gemm_mma(_p(x), _p(pieces), _p(logits), T, E, K, _stream()), "router_gemm_mma")
 
 
-ROUTE_SIGMOID_RAW, ROUTE_SIGMOID_RENORM, ROUTE_SOFTMAX_CHOSEN, ROUTE_SOFTMAX_ALL = 0, 1, 2, 3
+ROUTE_SIGMOID_RAW, ROUTE_SIGMOID_RENORM, ROUTE_SOFTMAX_CHOSEN, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID_SHARE = 0, 1, 2, 3, 4
 
 
 def router_topk(logits, bias, idx_out, w_out, renorm, scale: float) -> None:
@@ -439,7 +439,8 @@ def router_topk(logits, bias, idx_out, w_out, renorm, scale: float) -> None:
     (sigmoid scores as they are / divided by their sum; the bias enters the choice only), or
     ``ROUTE_SOFTMAX_CHOSEN``: the choice is by ``logit + bias`` and the weights are the softmax over the chosen
     values, or ``ROUTE_SOFTMAX_ALL``: the scores are the softmax over all logits, the choice is by ``score + bias``
-    and the weights are the chosen scores as they are."""
+    and the weights are the chosen scores as they are, or ``ROUTE_SIGMOID_SHARE``: sigmoid scores divided by their sum
+    also where one expert is chosen (True leaves a single score as it is)."""
     _want(logits, torch.float32, "logits"); _want(idx_out, torch.int32, "idx_out"); _want(w_out, torch.float32, "w_out")
     n_partials = 1 if logits.dim() == 2 else logits.shape[0]
     T, E = logits.shape[-2:]
@@ -1160,3 +1161,160 @@ def token_input(x, w_gate, table, offset: int, ids, out, status, gate=None) -> N
         raise ValueError("token_input: shape/dtype mismatch")
     _check(lib().qb_token_input_gate(_p(x), _p(w_gate), _p(table), table.shape[1], int(offset), _p(ids), _p(out),
                                      _code(out), T, W, D, table.shape[0], _p(status), _stream()), "token_input_gate")
+
+
+# ---- recurrences with one decay a (token, head) (csrc/decay_state.cu) ----------------------------------------------
+DECAY_MAX_DIM = 256           # key channels a head
+DECAY_CHUNK_MIN = 16          # portions of at least this many tokens run as chunks where the sizes allow
+
+
+class DecayGates:
+    """Where the decay and the weight of a (token, head) come from: ``DecayGates.constant(decay)`` (float32 ``[H]``,
+    weights of one), ``DecayGates.step(pre, bias, A_log)`` (``dt = softplus(pre + bias)``, decay ``exp(-exp(A_log) dt)``,
+    weight ``dt``; ``pre`` float32 ``[T, H]``, a column range of wider rows is fine) or ``DecayGates.given(log_decay,
+    weight)`` (float32 ``[T, H]``)."""
+
+    def __init__(self, kind: int, **tensors):
+        self.kind, self.t = kind, tensors
+
+    @classmethod
+    def constant(cls, decay):
+        # the logarithms of the float32 decays, taken in float64: both forms of the kernel use the same decay
+        return cls(0, decay=decay.contiguous(), log_decay=torch.log(decay.double()).clamp_min(-1e4).float().contiguous())
+
+    @classmethod
+    def step(cls, pre, bias, A_log):
+        return cls(1, step=pre, bias=bias, A_log=A_log)
+
+    @classmethod
+    def given(cls, log_decay, weight):
+        return cls(2, log_decay=log_decay, weight=weight)
+
+    def args(self, T: int, H: int):
+        t, null = self.t, ctypes.c_void_p(0)
+        for name, x in t.items():
+            _want(x, torch.float32, name)
+        if self.kind == 0:
+            if t["decay"].numel() != H:
+                raise ValueError("decay: one number a head is wanted")
+            return [0, _p(t["decay"]), _p(t["log_decay"]), null, 0, null, null, null]
+        if self.kind == 1:
+            pre = t["step"]
+            if tuple(pre.shape) != (T, H) or t["bias"].numel() != H or t["A_log"].numel() != H:
+                raise ValueError("step gates: shape mismatch")
+            ptr, stride = _rows_of(pre, H, "step")
+            return [1, null, null, ptr, stride, _p(t["bias"]), _p(t["A_log"]), null]
+        if t["log_decay"].numel() != T * H or t["weight"].numel() != T * H:
+            raise ValueError("given gates: one number a (token, head) is wanted")
+        return [2, null, _p(t["log_decay"]), null, 0, null, null, _p(t["weight"])]
+
+
+def memory_gates(proj, i_off: int, f_off: int, i_bias, f_bias, cap: float, m_state, req_start, req_slot, n_heads: int):
+    """Exponential gates with a running maximum per (request, head), from and into ``m_state`` ``[slots, heads]``:
+    ``i = cap tanh((x_i + b_i) / cap)``, ``f = logsigmoid(cap tanh((x_f + b_f) / cap))``, ``m' = max(f + m, i)``.
+    Returns float32 ``[T, heads]`` tensors ``(f + m - m', exp(i - m'), exp(-m'))``."""
+    for t, n in ((proj, "proj"), (i_bias, "i_bias"), (f_bias, "f_bias"), (m_state, "m_state")):
+        _want(t, torch.float32, n)
+    T, H = proj.shape[0], int(n_heads)
+    if (proj.stride(1) != 1 or min(i_off, f_off) < 0 or max(i_off, f_off) + H > proj.shape[1] or i_bias.numel() != H
+            or f_bias.numel() != H or tuple(m_state.shape[1:]) != (H,)):
+        raise ValueError("memory_gates: shape mismatch")
+    out = torch.empty((3, T, H), dtype=torch.float32, device=proj.device)
+    _check(lib().qb_memory_gates(ctypes.c_void_p(proj.data_ptr()), int(proj.stride(0)), int(i_off), int(f_off), _p(i_bias),
+                                 _p(f_bias), ctypes.c_float(cap), _p(m_state), _p(out[0]), _p(out[1]), _p(out[2]),
+                                 _p(req_start), _p(req_slot), T, req_slot.numel(), H, _stream()), "memory_gates")
+    return out[0], out[1], out[2]
+
+
+def rows_act(x, out, silu: bool = False) -> None:
+    """``out = x`` or ``silu(x)`` in the dtype of ``out``; ``x`` float32 ``[T, n]``, a column range of wider rows."""
+    T, n = x.shape
+    x_p, x_s = _rows_of(x, n, "x")
+    if tuple(out.shape) != (T, n):
+        raise ValueError("rows_act: shape mismatch")
+    _check(lib().qb_rows_act(x_p, ctypes.c_longlong(x_s), _p(out), _code(out), T, n, int(silu), _stream()), "rows_act")
+
+
+def decay_chunks_take(T: int, n_requests: int, longest: int, dim: int, vdim: int) -> bool:
+    """Whether a step of ``T`` tokens whose longest portion has ``longest`` (0: not known) is worth the chunk form, and
+    the sizes allow it."""
+    return (T > n_requests and (longest or T) >= DECAY_CHUNK_MIN
+            and bool(lib().qb_decay_chunks_supported(int(dim), int(vdim))))
+
+
+def decay_state(q, k, v, gates: DecayGates, state, out, req_start, req_slot, n_heads: int, n_groups: int, dim: int,
+                vdim: int, *, q_scale: float = 1.0, silu: bool = False, n_state=None, floor=None, den=None,
+                rows16=None, longest: int = 0, segments: bool | None = None) -> None:
+    """``S <- a S + w k v^T``, ``o = q_scale * S^T q`` per (request, head) over the step's tokens, from and into ``state``
+    float32 ``[slots, heads, dim, vdim]``; ``a``, ``w`` from ``gates``.  ``q``, ``k`` ``[T, groups * dim]`` (head h reads
+    group ``h // (heads / groups)``) and ``v`` ``[T, heads * vdim]`` are column ranges of rows with one stride, float32 or
+    bfloat16; ``silu``: they pass through it as they are read.  ``n_state`` float32 ``[slots, heads, dim]`` with ``floor``
+    and ``den`` float32 ``[T, heads]``: also ``n <- a n + w k`` and ``den = max(|q_scale n . q|, floor) + 1e-6``.
+    ``rows16``: the same q, k, v as bfloat16 (activated already, one stride): portions of ``DECAY_CHUNK_MIN`` tokens and
+    more then run in chunks on the tensor cores (``decay_chunks_take``); ``longest``: the step's longest portion if known.
+    ``segments`` False keeps them in one pass."""
+    T, H, G, D, E = q.shape[0], int(n_heads), int(n_groups), int(dim), int(vdim)
+    _want(state, torch.float32, "state"); _want(out, torch.float32, "out")
+    if (H % G or tuple(q.shape) != (T, G * D) or tuple(k.shape) != (T, G * D) or tuple(v.shape) != (T, H * E)
+            or out.numel() != T * H * E or tuple(state.shape[1:]) != (H, D, E)):
+        raise ValueError("decay_state: shape mismatch")
+
+    def rows(a, b, c):
+        if a.dtype != b.dtype or a.dtype != c.dtype or not (a.stride(0) == b.stride(0) == c.stride(0)) or \
+                not (a.stride(1) == b.stride(1) == c.stride(1) == 1) or not a.is_cuda:
+            raise ValueError("decay_state: q, k and v are columns of rows with one stride and dtype")
+        return [ctypes.c_void_p(t.data_ptr()) for t in (a, b, c)]
+
+    norm = [ctypes.c_void_p(0)] * 3
+    if n_state is not None:
+        for t, n in ((n_state, "n_state"), (floor, "floor"), (den, "den")):
+            _want(t, torch.float32, n)
+        if tuple(n_state.shape[1:]) != (H, D) or floor.numel() != T * H or den.numel() != T * H:
+            raise ValueError("decay_state: shape mismatch of the normaliser")
+        norm = [_p(n_state), _p(floor), _p(den)]
+    R = req_slot.numel()
+    g = gates.args(T, H)
+    most = 0x7fffffff
+    if rows16 is not None:
+        if rows16[0].dtype != torch.bfloat16 or [tuple(t.shape) for t in rows16] != [tuple(t.shape) for t in (q, k, v)]:
+            raise ValueError("decay_state: rows16 are bfloat16 rows of the same sizes")
+        fn = lib().qb_decay_chunks_scratch
+        fn.restype = ctypes.c_longlong
+        n = int(fn(T, R, H, D, E, int(n_state is not None))) if segments is not False else 0
+        scratch = torch.empty(n, dtype=torch.float32, device=q.device) if n else None
+        _check(lib().qb_decay_chunks(*rows(*rows16), ctypes.c_longlong(rows16[0].stride(0)), *g, _p(state), *norm, _p(out),
+                                     _p(scratch), _p(req_start), _p(req_slot), T, R, H, G, D, E, ctypes.c_float(q_scale),
+                                     DECAY_CHUNK_MIN, _stream()), "decay_chunks", 4 if n else 1)
+        if R == 1 and T >= DECAY_CHUNK_MIN:
+            return
+        most = DECAY_CHUNK_MIN - 1
+    _check(lib().qb_decay_chain(*rows(q, k, v), _code(q), ctypes.c_longlong(q.stride(0)), *g, _p(state), *norm, _p(out),
+                                _p(req_start), _p(req_slot), T, R, H, G, D, E, ctypes.c_float(q_scale), int(silu), most,
+                                _stream()), "decay_chain")
+
+
+def decay_out(o, gate, gain, out, n_heads: int, vdim: int, parts: int, eps: float, *, den=None, x=None, skip=None,
+              gate_first: bool = False) -> None:
+    """From a recurrence's results ``o`` float32 ``[T, heads, vdim]`` to the rows its output projection reads:
+    ``y = o / den + skip[h] * x`` (``den`` float32 ``[T, heads]``; ``skip`` float32 ``[heads]`` with ``x`` ``[T, heads *
+    vdim]`` in the dtype of ``out``; both optional), then ``gate_first``: ``y * silu(gate)``, normed in ``parts`` equal
+    parts of the row, times ``gain`` (``[heads * vdim]``); else normed in parts, times ``gain``, times ``sigmoid(gate)``.
+    ``gate`` float32 ``[T, heads * vdim]``, a column range of wider rows."""
+    T, C = out.shape
+    _want(o, torch.float32, "o"); _want(gain, torch.float32, "gain")
+    if C != n_heads * vdim or o.numel() != T * C or gain.numel() != C or tuple(gate.shape) != (T, C) or C % parts:
+        raise ValueError("decay_out: shape mismatch")
+    g_p, g_s = _rows_of(gate, C, "gate")
+    x_p, x_s = ctypes.c_void_p(0), 0
+    if skip is not None:
+        _want(skip, torch.float32, "skip")
+        if x is None or tuple(x.shape) != (T, C) or x.dtype != out.dtype or x.stride(1) != 1 or skip.numel() != n_heads:
+            raise ValueError("decay_out: the skipped rows do not fit")
+        x_p, x_s = ctypes.c_void_p(x.data_ptr()), int(x.stride(0))
+    if den is not None:
+        _want(den, torch.float32, "den")
+        if den.numel() != T * n_heads:
+            raise ValueError("decay_out: one denominator a (token, head) is wanted")
+    _check(lib().qb_decay_out(_p(o), _p(den), x_p, ctypes.c_longlong(x_s), _p(skip), g_p, ctypes.c_longlong(g_s), _p(gain),
+                              _p(out), _code(out), T, int(n_heads), int(vdim), int(parts), ctypes.c_float(eps),
+                              int(gate_first), _stream()), "decay_out")

@@ -1,2 +1,2 @@
 """Architectures: each module maps a configuration to a model specification and registers itself."""
-from . import guravik, lotilix, minimax_m3, puvolix, tarulix, tirizen  # noqa: F401
+from . import gedelorn, guravik, lotilix, minimax_m3, puvolix, tarulix, tirizen  # noqa: F401

@@ -6,6 +6,8 @@ index); weights are the bias-free scores, renormalised (``+ 1e-20``) and scaled;
 ``down(silu(gate x) * up x)`` (``w1`` gate, ``w3`` up, ``w2`` down); the weight is applied after
 ``down``; the k results are summed in float32 in slot order.  No shared expert.
 
+``sigmoid_ungated_experts``: the same scores, always divided by their sum, with ungated experts and a shared one.
+
 ``softmax_topk_experts`` shares the plan and the kernels: the router has a bias that is part of the logits
 (``z = gate x + bias``, float32), the ``top_k`` largest logits choose, the weights are the softmax over the
 chosen logits only, and an expert is ungated, ``down(relu(up x)^2)``.
@@ -332,3 +334,33 @@ class InputWeightedExperts(SigmoidTopKExperts):
         routed = super().forward
         extra, y = run_beside(lambda: self.shared.forward(x, ctx), lambda: routed(x, ctx), x.device)
         return Addends(y, extra=extra.y if isinstance(extra, Addends) else extra)
+
+
+@register("feed_forward", "sigmoid_ungated_experts")
+class SigmoidUngatedExperts(SoftmaxTopKExperts):
+    """Sigmoid-routed ungated experts: router logits float32, scores ``sigmoid``, the ``top_k`` largest chosen (the lower
+    index among equals), the weights the chosen scores divided by their sum (``+ 1e-20``; also where one is chosen) times
+    ``scaling``; an expert is ``down(relu(up x)^2)`` without biases.  ``shared_size`` > 0: an expert of the same form and
+    that inner size that every token passes is added.  ``names``: gate (the router), templates up / down with ``{e}`` and
+    shared_up / shared_down.  Returns the routed slots with the shared expert's output as a second addend, for a block
+    that norms the sum."""
+
+    def __init__(self, hidden_size: int, expert_size: int, n_experts: int, top_k: int, scaling: float, names: dict,
+                 shared_size: int = 0):
+        super().__init__(hidden_size, expert_size, n_experts, top_k, use_bias=False, names=names)
+        self.renorm, self.scaling = kernels.ROUTE_SIGMOID_SHARE, float(scaling)
+        self.shared_size = int(shared_size)
+        self.shared = None
+        if self.shared_size:
+            from .dense import UngatedDense
+            self.shared = UngatedDense(hidden_size, shared_size, {"up": names["shared_up"], "down": names["shared_down"]})
+
+    def children(self):
+        return [self.shared] if self.shared is not None else []
+
+    def forward(self, x, ctx):
+        if self.shared is None:
+            return Addends(super().forward(x, ctx))
+        routed = super().forward
+        extra, y = run_beside(lambda: self.shared.forward(x, ctx), lambda: routed(x, ctx), x.device)
+        return Addends(y, extra=extra)

@@ -12,15 +12,18 @@ from .base import Addends, Norm, NormedPending, StreamCopy, StreamsPending, Tens
 class RMSNorm(Norm):
     graph_safe = True
 
-    """``weight * x * rsqrt(mean(x^2) + eps)`` with float32 statistics; plain weight (no ``1 + w``)."""
+    """``weight * x * rsqrt(mean(x^2) + eps)`` with float32 statistics."""
 
-    def __init__(self, width: int, eps: float, weight_name: str, scalar_gain: bool = False, groups: int = 1):
+    def __init__(self, width: int, eps: float, weight_name: str, scalar_gain: bool = False, groups: int = 1,
+                 around_zero: bool = False):
         """``scalar_gain``: the checkpoint holds ONE number that multiplies every coordinate (a tensor without
         dimensions); it is spread over ``width`` gains at load, so the kernels see the usual vector.  ``groups``:
         the vector is cut into that many equal consecutive parts and each is divided by its OWN root mean square
-        (``eps`` inside each root); the gain still has ``width`` numbers."""
+        (``eps`` inside each root); the gain still has ``width`` numbers.  ``around_zero``: the checkpoint holds the
+        gain minus one; the one is added at load, in float32."""
         self.width, self.eps, self.weight_name = int(width), float(eps), weight_name
         self.scalar_gain = bool(scalar_gain)
+        self.around_zero = bool(around_zero)
         self.groups = int(groups)
         if not 1 <= self.groups <= kernels.NORM_MAX_GROUPS or self.width % self.groups:
             raise ValueError(f"rms_norm: {groups} groups do not divide a width of {width} "
@@ -28,10 +31,13 @@ class RMSNorm(Norm):
         self.weight: torch.Tensor | None = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.weight_name, () if self.scalar_gain else (self.width,), kind="f32", init="gain")]
+        return [TensorSpec(self.weight_name, () if self.scalar_gain else (self.width,), kind="f32",
+                           init="bias" if self.around_zero else "gain")]
 
     def load(self, fetch):
         self.weight = fetch(self.weight_name)
+        if self.around_zero:
+            self.weight = self.weight + 1.0
         if self.scalar_gain:
             self.weight = self.weight.reshape(1).expand(self.width).contiguous()
 

@@ -21,6 +21,10 @@ Each extra is a parameter and is off unless it is given:
 * ``value_blend``: ``"source"``: the layer leaves its values (per token of the step, float32) under ``blend_key``
   for later layers; ``"blend"``: its values become ``(1 - lambda) v + lambda v_source`` with the learned number
   ``vmix`` before they are cached.  A source layer has no fraction of its own.
+* ``values_from_keys``: the values are the projected keys (bias included) before norm and rotation; there is no ``v``
+  tensor and the head sizes are equal.
+
+With ``biases`` a projection has a bias where ``names`` gives it one (``q_b``, ``k_b``, ``v_b``, ``o_b``).
 
 Scores, softmax weights, the bias, the sink and the mixing of heads are float32; the projections' float32
 accumulators (with the biases) feed the kernel that norms, rotates and fills the cache.
@@ -58,7 +62,7 @@ class WindowAttention(Mixer):
                  norm_eps: float, names: dict, value_dim: int | None = None, position=("none", {}),
                  unit_qk: bool = False, biases: bool = False, distance_bias: tuple | None = None, sink: bool = False,
                  softcap: float = 0.0, pool: int = 0, talk: bool = False, value_blend: str | None = None,
-                 blend_key: str = "blend_values"):
+                 blend_key: str = "blend_values", values_from_keys: bool = False):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} q heads are not a multiple of {n_kv_heads} kv heads")
         value_dim = head_dim if value_dim is None else int(value_dim)
@@ -79,8 +83,12 @@ class WindowAttention(Mixer):
                                                (self.distance_bias[0] > 1 and self.distance_bias[1] <= self.distance_bias[0] // 2)):
             raise ValueError(f"distance_bias {self.distance_bias}: the ladder must end beyond its first half")
         self.value_blend, self.blend_key = value_blend, blend_key
+        self.tied_v = bool(values_from_keys)
+        if self.tied_v and (value_dim != head_dim or value_blend is not None):
+            raise ValueError("window_attention: values that are the keys have the keys' size and are not blended")
         self.position = make("position", position) if isinstance(position, tuple) else position
-        self.names = dict(names)     # q, k, v, o (+ ".b" names q_b, k_b, v_b, o_b), rel, sink, talk, vmix
+        self.names = dict(names)     # q, k, v, o (and their biases q_b, k_b, v_b, o_b), rel, sink, talk, vmix
+        self.biased = {s for s in ("q", "k", "v", "o") if self.biases and s + "_b" in self.names and not (s == "v" and self.tied_v)}
         self.w_qkv = self.w_o = self.b_qkv = self.b_o = self.dist_table = self.sink = self.talk = self.lam = None
 
     def children(self):
@@ -88,11 +96,12 @@ class WindowAttention(Mixer):
 
     def tensor_specs(self):
         n, W, hd, vd = self.names, self.hidden, self.hd, self.vd
-        specs = [TensorSpec(n["q"], (self.nq * hd, W)), TensorSpec(n["k"], (self.nkv * hd, W)),
-                 TensorSpec(n["v"], (self.nkv * vd, W)), TensorSpec(n["o"], (W, self.nq * vd))]
-        if self.biases:
-            specs += [TensorSpec(n["q_b"], (self.nq * hd,), "f32", "bias"), TensorSpec(n["k_b"], (self.nkv * hd,), "f32", "bias"),
-                      TensorSpec(n["v_b"], (self.nkv * vd,), "f32", "bias"), TensorSpec(n["o_b"], (W,), "f32", "bias")]
+        specs = [TensorSpec(n["q"], (self.nq * hd, W)), TensorSpec(n["k"], (self.nkv * hd, W)), TensorSpec(n["o"], (W, self.nq * vd))]
+        if not self.tied_v:
+            specs.append(TensorSpec(n["v"], (self.nkv * vd, W)))
+        for s, size in (("q", self.nq * hd), ("k", self.nkv * hd), ("v", self.nkv * vd), ("o", W)):
+            if s in self.biased:
+                specs.append(TensorSpec(n[s + "_b"], (size,), "f32", "bias"))
         if self.distance_bias is not None:
             specs.append(TensorSpec(n["rel"], (self.distance_bias[0], self.nq), "f32", "bias"))
         if self.value_blend == "blend":
@@ -108,17 +117,22 @@ class WindowAttention(Mixer):
         q = fetch(n["q"])
         a = self.nq * self.hd
         b = a + self.nkv * self.hd
-        c = b + self.nkv * self.vd
+        c = b + (0 if self.tied_v else self.nkv * self.vd)
         # one fused input projection, its rows padded to a multiple of 8 (every product row starts on 16 bytes)
         rows = -(-c // 8) * 8
         self.w_qkv = torch.zeros((rows, self.hidden), dtype=q.dtype, device=q.device)
         self.w_qkv[:a].copy_(q)
         del q
         self.w_qkv[a:b].copy_(fetch(n["k"]))
-        self.w_qkv[b:c].copy_(fetch(n["v"]))
+        if not self.tied_v:
+            self.w_qkv[b:c].copy_(fetch(n["v"]))
         self.w_o = fetch(n["o"])
-        if self.biases:
-            self.b_qkv = torch.cat([fetch(n["q_b"]), fetch(n["k_b"]), fetch(n["v_b"])]).contiguous()
+        if self.biased - {"o"}:
+            self.b_qkv = torch.zeros(c, dtype=torch.float32, device=self.w_qkv.device)
+            for s, lo, hi in (("q", 0, a), ("k", a, b), ("v", b, c)):
+                if s in self.biased:
+                    self.b_qkv[lo:hi].copy_(fetch(n[s + "_b"]))
+        if "o" in self.biased:
             self.b_o = fetch(n["o_b"]).contiguous()
         if self.distance_bias is not None:
             rel = fetch(n["rel"])
@@ -163,7 +177,7 @@ class WindowAttention(Mixer):
             qkv, q, cache.k, cache.v, None, None, kernels.NORM_PER_HEAD if self.unit_qk else kernels.NORM_NONE, self.eps,
             inv_freq, pair_axis, ctx.positions, ctx.tok_pos, ctx.tok_req, cache.tables["k"], self.nq, self.nkv, self.hd,
             rd, cache.page_size, ctx.status, vd=self.vd, bias=self.b_qkv, v_first=v_first, v_lambda=self.lam,
-            v_export=v_export)
+            v_export=v_export, interleaved=bool(getattr(self.position, "interleaved", False)), tied_values=self.tied_v)
         pooled = {}
         if self.pool:
             kp, vp = cache.streams["k_pooled"], cache.streams["v_pooled"]
@@ -179,4 +193,4 @@ class WindowAttention(Mixer):
                                  softcap=self.softcap, talk=self.talk, scratch=scratch,
                                  n_requests=int(ctx.req_start.numel()) - 1, **pooled)
         y = linear(out.view(T, self.nq * self.vd), self.w_o, out_dtype=torch.float32)
-        return Addends(y, bias=self.b_o) if self.biases else y
+        return Addends(y, bias=self.b_o) if self.b_o is not None else y

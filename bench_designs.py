@@ -1,4 +1,4 @@
-"""``bench.py --design guravik`` / ``--design tirizen`` / ``--design tarulix`` / ``--design puvolix`` / ``--design lotilix``: another decoder beside the MiniMax-M3 decoder at equal sizes.
+"""``bench.py --design guravik`` / ``--design tirizen`` / ``--design tarulix`` / ``--design puvolix`` / ``--design lotilix`` / ``--design gedelorn``: another decoder beside the MiniMax-M3 decoder at equal sizes.
 
 For a few sizes that resemble a real model's layers (seeded random weights, bfloat16): one prompt of
 ``--prompt-len`` tokens as one step (tokens a second) and decode steps of ``--batch`` requests at that
@@ -42,6 +42,14 @@ channel, dense feed-forwards; given a feed-forward in every layer here), and Min
 latent attention beside Guravik's form of it, the chunked attention beside Puvolix's form of the same kernels, the
 recurrence beside Puvolix's (one decay a head) and Guravik's ``delta_rule``, and the launches around the token's own input
 beside ``normed_add_rmsnorm``.
+
+``--design gedelorn``: the Gedelorn decoder (layers: a state-space recurrence with one decay a head and a dense feed-forward,
+windowed attention with capped scores beside constant-decay linear attention and a matrix memory, both with routed ungated
+experts and a shared one; norms before and after each sublayer) beside Tarulix, the closest existing model (windowed
+attention beside a selective scan, normed outputs, routed and shared experts), and MiniMax-M3, all at equal sizes.  Alone: the
+recurrence in its three uses beside Tarulix's ``selective_scan``, Tirizen's ``gla`` and Puvolix's ``gated_delta``; the attention
+in the form Gedelorn runs it beside Tarulix's biased form; the exponential gates and the launch between recurrence and output
+projection beside ``head_norm_gate``.
 """
 
 from __future__ import annotations
@@ -420,7 +428,7 @@ def run_tirizen(args) -> dict:
 def window_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int, hd: int, window: int, kind: str,
                 pool: int = 64, page: int = 16) -> dict:
     """``window_attention`` alone: ``reqs`` requests whose last ``tokens_per_req`` tokens (ending at ``context``) are
-    the step.  ``kind`` "biased": distance bias and sink; "pooled": score cap, pooled blocks and mixed head weights
+    the step.  ``kind`` "biased": distance bias and sink; "capped": a score cap alone; "pooled": score cap, pooled blocks and mixed head weights
     (with the second launch that mixes).  Flops count ``4 * head_dim`` a (query head, visible key), pooled rows too;
     bytes count the visible keys and values once a request."""
     import torch
@@ -442,6 +450,8 @@ def window_attn(tokens_per_req: int, reqs: int, context: int, nq: int, nkv: int,
     extras = {}
     if kind == "biased":
         extras = dict(dist_bias=torch.randn(window, nq, device=dev), sink=torch.zeros(nq, device=dev))
+    elif kind == "capped":
+        extras = dict(softcap=30.0)
     else:
         rows = -(-context // pool)
         ppp = -(-rows // page)
@@ -746,6 +756,160 @@ def scan(tokens_per_req: int, reqs: int, inner: int, N: int, rank: int) -> dict:
             "GB/s": round(nbytes / ms / 1e6, 1), "fp32 TFLOP/s": round(flops / ms / 1e9, 2)}
 
 
+GEDELORN_SIZES = {
+    "w2048": dict(width=2048, groups=2, vocab=32000, ff=5632, attn_heads=16, dim=128, window=1024, ssm_heads=64, ssm_vdim=64, state=128,
+                  ssm_groups=8, lin_heads=16, lin_dim=128, mem_heads=8, mem_dim=128, mem_vdim=256,
+                  pool=64, rot=64, inner=4096, scan_state=16, dt_rank=128, taps=4),
+    "w4096": dict(width=4096, groups=2, vocab=32000, ff=11008, attn_heads=32, dim=128, window=1024, ssm_heads=128, ssm_vdim=64, state=128,
+                  ssm_groups=8, lin_heads=32, lin_dim=128, mem_heads=8, mem_dim=256, mem_vdim=512,
+                  pool=64, rot=64, inner=8192, scan_state=16, dt_rank=256, taps=4),
+}
+
+
+def gedelorn_raw(s: dict) -> dict:
+    """Per group of three layers: the state-space mixer with a dense feed-forward, the parallel mixer and the matrix memory with
+    8 routed ungated experts of which 2 are chosen and a shared one, together as wide as ``ff``."""
+    moe = {"kind": "moe", "expert": {"ff": 3 * s["ff"] // 8}, "router": {"experts": 8, "top": 2, "scale": 1.5}, "shared": {"ff": s["ff"] // 4}}
+    ssm = {"heads": s["ssm_heads"], "vdim": s["ssm_vdim"], "state": s["state"], "groups": s["ssm_groups"], "conv": s["taps"],
+           "norm_groups": s["ssm_groups"]}
+    left = {"heads": s["attn_heads"], "kv_heads": max(1, s["attn_heads"] // 4), "dim": s["dim"], "vdim": s["dim"],
+            "scale": 1.0 / math.sqrt(s["dim"]), "softcap": 30.0, "mask": {"size": s["window"]}, "rot": {"dims": s["dim"], "base": 1e6}}
+    H = s["lin_heads"]
+    right = {"heads": H, "dim": s["lin_dim"], "vdim": s["lin_dim"], "decay": [math.exp(-(2.0 ** (-8.0 * (h + 1) / H))) for h in range(H)]}
+    par = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 1.1}
+    mem = {"heads": s["mem_heads"], "dim": s["mem_dim"], "vdim": s["mem_vdim"], "gate_cap": 15.0}
+    layers = [{"type": "mamba2", "mixer": ssm, "mlp": {"kind": "dense", "ff": s["ff"]}}, {"type": "parallel", "mixer": par, "mlp": moe},
+              {"type": "mlstm", "mixer": mem, "mlp": moe}] * s["groups"]
+    return {"architecture": "Gedelorn", "vocab": s["vocab"], "width": s["width"], "layers": layers, "norm": {"eps": 1e-5}}
+
+
+def decay_state(tokens_per_req: int, reqs: int, H: int, G: int, D: int, E: int, kind: str) -> dict:
+    """The recurrence ``decay_state`` alone in one of its three uses: ``step`` (state-space mixer; bfloat16 rows from the
+    convolution), ``constant`` and ``memory`` (with a normaliser; both read float32 rows for single tokens, bfloat16 rows for
+    prompts).  Bytes: the state read and written, q, k and v (q and k of a group once), the outputs and the gates."""
+    import torch
+    import bench_kernels as bk
+    from quanta_b200 import kernels as k
+    dev = bk.DEV
+    T, single = tokens_per_req * reqs, tokens_per_req == 1
+    n = 2 * G * D + H * E
+    dtype = torch.float32 if single and kind != "step" else torch.bfloat16
+    x = torch.randn(T, n, device=dev).to(dtype)
+    qkv = x[:, : G * D], x[:, G * D: 2 * G * D], x[:, 2 * G * D:]
+    if kind == "step":
+        gates = k.DecayGates.step(torch.randn(T, H, device=dev), torch.zeros(H, device=dev), torch.zeros(H, device=dev))
+    elif kind == "constant":
+        gates = k.DecayGates.constant(torch.full((H,), 0.98, device=dev))
+    else:
+        gates = k.DecayGates.given(-torch.rand(T, H, device=dev), torch.rand(T, H, device=dev))
+    layers = 1 if not single else max(1, min(16, int(2e9 // (reqs * H * D * E * 4))))
+    states = [(torch.zeros(reqs, H, D, E, device=dev), torch.zeros(reqs, H, D, device=dev)) for _ in range(layers)]
+    out = torch.empty(T, H, E, device=dev)
+    floor, den = torch.ones(T, H, device=dev), torch.empty(T, H, device=dev)
+    starts = torch.arange(0, T + 1, tokens_per_req, dtype=torch.int32, device=dev)
+    slots = torch.arange(reqs, dtype=torch.int32, device=dev)
+
+    def all_layers():
+        for s, n_s in states:
+            k.decay_state(*qkv, gates, s, out, starts, slots, H, G, D, E, silu=kind == "constant" and single, longest=tokens_per_req,
+                          rows16=None if single else qkv, **(dict(n_state=n_s, floor=floor, den=den) if kind == "memory" else {}))
+    ms = (bk.timed_graph(all_layers, reps=1) if single else bk.timed(all_layers, n=5, warm=2)) / layers
+    nbytes = 2 * reqs * H * D * E * 4 + T * (n * x.element_size() + H * E * 4 + (0 if kind == "constant" else H * 4))
+    if kind == "memory":
+        nbytes += 2 * reqs * H * D * 4 + T * H * 12
+    # what the recurrence itself needs, token by token: the state's update and its read
+    return {"kernel": f"decay_state ({kind})", "requests": reqs, "tokens_per_request": tokens_per_req, "heads": H, "groups": G, "dim": D,
+            "vdim": E, "layers": layers, "us": round(ms * 1e3, 2), "tokens/s": round(T / ms * 1e3, 1),
+            "GB/s": round(nbytes / ms / 1e6, 1), "token-by-token TFLOP/s": round(5.0 * D * E * H * T / ms / 1e9, 2)}
+
+
+def around_the_recurrence(tokens: int, H: int, D: int, E: int) -> dict:
+    """The exponential gates, the rows' rounding, and the launch between recurrence and output projection (a norm a head; a
+    norm over the whole row; a gate before a norm in eight parts) beside ``head_norm_gate``."""
+    import torch
+    import bench_kernels as bk
+    from quanta_b200 import kernels as k
+    dev = bk.DEV
+    T, C = tokens, H * E
+    proj = torch.randn(T, 2 * H * D + 2 * C + 2 * H, device=dev)
+    o, out, act = torch.randn(T, H, E, device=dev), torch.empty(T, C, device=dev, dtype=torch.bfloat16), \
+        torch.empty(T, 2 * H * D + C, device=dev, dtype=torch.bfloat16)
+    gain, den, skip = torch.ones(C, device=dev), torch.ones(T, H, device=dev), torch.ones(H, device=dev)
+    gate = proj[:, 2 * H * D + C: 2 * H * D + 2 * C]
+    m, b = torch.zeros(1, H, device=dev), torch.zeros(H, device=dev)
+    starts, slot = torch.tensor([0, T], dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+    x = out.clone()
+    runs = {"memory_gates": (lambda: k.memory_gates(proj, 2 * H * D + 2 * C, 2 * H * D + 2 * C + H, b, b, 15.0, m, starts, slot, H), T * H * 20),
+            "rows_act": (lambda: k.rows_act(proj[:, : 2 * H * D + C], act, silu=True), T * (2 * H * D + C) * 6),
+            "decay_out (a norm a head)": (lambda: k.decay_out(o, gate, gain, out, H, E, H, 1e-5, den=den), T * C * 10),
+            "decay_out (one norm)": (lambda: k.decay_out(o, gate, gain, out, H, E, 1, 1e-5), T * C * 10),
+            "decay_out (gate, norm in 8 parts)": (lambda: k.decay_out(o, gate, gain, out, H, E, 8, 1e-5, x=x, skip=skip, gate_first=True), T * C * 12),
+            "head_norm_gate": (lambda: k.head_norm_gate(o, proj, 2 * H * D + C, gain, out, H, E, 1e-5), T * C * 10)}
+    res = {"tokens": T, "heads": H, "dim": D, "vdim": E}
+    for name, (fn, nbytes) in runs.items():
+        ms = bk.timed_graph(fn, reps=20) if T <= 64 else bk.timed(fn, n=5, warm=2)
+        res[name] = {"us": round(ms * 1e3, 2), "GB/s": round(nbytes / ms / 1e6, 1)}
+    return res
+
+
+def run_gedelorn(args) -> dict:
+    import bench
+    from quanta_b200.config import GedelornConfig, MiniMaxM3Config, TarulixConfig
+    pk, pk_src = bench.peaks()
+    clocks = bench.ClockSampler()
+    clocks.start()
+    models = {}
+    for name, s in GEDELORN_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        t0 = time.time()
+        g = _model_numbers(GedelornConfig.from_dict(gedelorn_raw(s)), args.prompt_len, args.batch, args.steps, args.warmup)
+        t = _model_numbers(TarulixConfig.from_dict(tarulix_raw(dict(s, state=s["scan_state"]))), args.prompt_len, args.batch, args.steps, args.warmup)
+        m = _model_numbers(MiniMaxM3Config.from_dict(minimax_raw(s)), args.prompt_len, args.batch, args.steps, args.warmup)
+        models[name] = {"sizes": s, "gedelorn": g, "tarulix": t, "minimax_m3": m}
+        print(f"[bench] {name}: gedelorn {g}\n[bench] {name}: tarulix {t}\n[bench] {name}: minimax_m3 {m} ({time.time() - t0:.0f} s)",
+              file=sys.stderr, flush=True)
+    s = GEDELORN_SIZES["w2048"]
+    T, B = args.prompt_len, args.batch
+    tensor, hbm = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+    uses = {"step": (s["ssm_heads"], s["ssm_groups"], s["state"], s["ssm_vdim"]), "constant": (s["lin_heads"], s["lin_heads"], s["lin_dim"], s["lin_dim"]),
+            "memory": (s["mem_heads"], s["mem_heads"], s["mem_dim"], s["mem_vdim"])}
+    prompt = {kind: decay_state(T, 1, *size, kind) for kind, size in uses.items()}
+    prompt.update({f"{kind}, 8 prompts of {T // 4}": decay_state(T // 4, 8, *size, kind) for kind, size in uses.items()})
+    one = {kind: decay_state(1, B, *size, kind) for kind, size in uses.items()}
+    one.update({f"{kind}, batch 64": decay_state(1, 64, *size, kind) for kind, size in uses.items()})
+    prompt.update(tarulix_scan=scan(T, 1, s["inner"], s["scan_state"], s["dt_rank"]), tirizen_gla=gla(T, 1, 16, 128, 128),
+                  puvolix_gated_delta=gated_delta(T, 1, 16, 8, 128, 128))
+    one.update(tarulix_scan=scan(1, B, s["inner"], s["scan_state"], s["dt_rank"]), tirizen_gla=gla(1, B, 16, 128, 128),
+               puvolix_gated_delta=gated_delta(1, B, 16, 8, 128, 128))
+    for r in [*prompt.values(), *one.values()]:
+        r["frac_of_copy_bandwidth"] = round(r["GB/s"] * 1e9 / hbm, 4)
+    Hq, Hk, hd, W = s["attn_heads"], max(1, s["attn_heads"] // 4), s["dim"], s["window"]
+    wp = {kind: window_attn(T, 1, T, Hq, Hk, hd, W, kind) for kind in ("capped", "biased")}
+    wd = {kind: window_attn(1, B, 4 * T, Hq, Hk, hd, W, kind) for kind in ("capped", "biased")}
+    for r in wp.values():
+        r["frac_of_tensor_peak"] = round(r["TFLOP/s"] * 1e12 / tensor, 4)
+    for r in wd.values():
+        r["frac_of_copy_bandwidth"] = round(r["GB/s"] * 1e9 / hbm, 4)
+    ap, ad = (around_the_recurrence(n, s["mem_heads"], s["mem_dim"], s["mem_vdim"]) for n in (T, B))
+    for r in (ap, ad):
+        for v in r.values():
+            if isinstance(v, dict):
+                v["frac_of_copy_bandwidth"] = round(v["GB/s"] * 1e9 / hbm, 4)
+    kernels_alone = {"recurrence_prompt": prompt, "recurrence_single_tokens": one, "window_attention_prompt": wp,
+                     "window_attention_single_tokens": wd, "around_the_recurrence_prompt": ap, "around_the_recurrence_single_tokens": ad}
+    for k_, v in kernels_alone.items():
+        for n_, r in v.items():
+            print(f"[bench] {k_}: {n_}: {r}", file=sys.stderr, flush=True)
+    first = next(iter(models.values()))["gedelorn"] if models else {}
+    return {"metric": f"Gedelorn decode tokens/s (batch {args.batch}, {args.prompt_len}-token prompts) beside Tarulix and MiniMax-M3 at equal sizes",
+            "value": first.get("decode_tok_s"), "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "ms_per_step": first.get("decode_ms"), "higher_is_better": True, "dtype": "bf16",
+            "data": "synthetic (seeded uniform token ids, seeded random weights)", "design": "gedelorn", "models": models,
+            "kernels": kernels_alone, "peaks": {**pk, "source": pk_src}, "clocks": clocks.stop(),
+            "gpu_launches": first.get("launches_per_decode_step", 0) * args.steps, "impl": "ours"}
+
+
 def run_tarulix(args) -> dict:
     import bench
     import bench_kernels as bk
@@ -801,6 +965,8 @@ def run(args) -> dict:
         return run_puvolix(args)
     if getattr(args, "design", "guravik") == "lotilix":
         return run_lotilix(args)
+    if getattr(args, "design", "guravik") == "gedelorn":
+        return run_gedelorn(args)
     import torch
     import bench
     import bench_kernels as bk
@@ -851,8 +1017,8 @@ if __name__ == "__main__":
     import argparse
     ap = argparse.ArgumentParser()
     ap.add_argument("kernel", choices=["latent_prefill", "latent_decode", "delta_rule", "gla", "streams_norm", "window_prefill",
-                                       "window_decode", "scan"])
-    ap.add_argument("--kind", default="biased", choices=["biased", "pooled"])
+                                       "window_decode", "scan", "decay_state"])
+    ap.add_argument("--kind", default="biased", choices=["biased", "capped", "pooled", "step", "constant", "memory"])
     ap.add_argument("--window", type=int, default=1024)
     ap.add_argument("--tokens", type=int, default=2048)
     ap.add_argument("--batch", type=int, default=8)
@@ -860,6 +1026,8 @@ if __name__ == "__main__":
     ap.add_argument("--latent", type=int, default=256)
     ap.add_argument("--rot", type=int, default=64)
     ap.add_argument("--dim", type=int, default=64)
+    ap.add_argument("--vdim", type=int, default=0)
+    ap.add_argument("--groups", type=int, default=0)
     a = ap.parse_args()
     if a.kernel == "latent_prefill":
         print(json.dumps(latent_prefill(a.tokens, a.heads, a.latent, a.rot)))
@@ -873,6 +1041,8 @@ if __name__ == "__main__":
         print(json.dumps(window_attn(a.tokens, 1, a.tokens, a.heads, max(1, a.heads // 4), 128, a.window, a.kind)))
     elif a.kernel == "window_decode":
         print(json.dumps(window_attn(1, a.batch, a.tokens, a.heads, max(1, a.heads // 4), 128, a.window, a.kind)))
+    elif a.kernel == "decay_state":
+        print(json.dumps(decay_state(a.tokens, a.batch, a.heads, a.groups or a.heads, a.dim, a.vdim or a.dim, a.kind)))
     elif a.kernel == "scan":
         print(json.dumps(scan(a.tokens, a.batch, 4096, 16, 128)))
     else:

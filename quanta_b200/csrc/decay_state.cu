@@ -65,7 +65,7 @@ __device__ __forceinline__ void ds_log_gate(const DsGates& g, int t, int h, int 
 // ---------------------------------------------------------------------------------------------
 // exponential gates
 // ---------------------------------------------------------------------------------------------
-constexpr int DS_GATE_RUN = 8;        // tokens a thread walks
+constexpr int DS_GATE_RUN = 2;        // tokens a thread walks
 
 __device__ __forceinline__ void ds_raw_gates(const float* __restrict__ proj, int stride, int i_off, int f_off, int t,
                                              int h, float bi, float bf, float cap, float& i, float& f) {
@@ -135,13 +135,40 @@ __global__ void memory_gates_kernel(const float* __restrict__ proj, int stride, 
   if (tid == 0) *m_at = (float)m_in;
 }
 
+// The same for a step of single tokens: a thread a (request, head), the same numbers without the scan.
+__global__ void memory_gates_single_kernel(const float* __restrict__ proj, int stride, int i_off, int f_off,
+                                           const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
+                                           float* __restrict__ m_state, float* __restrict__ log_decay,
+                                           float* __restrict__ weight, float* __restrict__ floor_out,
+                                           const int* __restrict__ req_slot, int R, int H) {
+  const int at = blockIdx.x * blockDim.x + threadIdx.x;        // token r of request r
+  if (at >= R * H) return;
+  const int r = at / H, h = at % H;
+  float* m_at = m_state + (size_t)req_slot[r] * H + h;
+  float iv, fv;
+  ds_raw_gates(proj, stride, i_off, f_off, r, h, i_bias[h], f_bias[h], cap, iv, fv);
+  const double before = (double)*m_at, m = fmax((double)fv + before, (double)iv);
+  const float now = (float)m;
+  log_decay[at] = (float)((double)fv + before - (double)now);
+  weight[at] = expf((float)((double)iv - (double)now));
+  floor_out[at] = expf(-now);
+  *m_at = now;
+}
+
 extern "C" int qb_memory_gates(const float* proj, int stride, int i_off, int f_off, const float* i_bias,
                                const float* f_bias, float cap, float* m_state, float* log_decay, float* weight,
                                float* floor_out, const int* req_start, const int* req_slot, int T, int R, int H,
                                cudaStream_t stream) {
   if (T <= 0 || R <= 0) return 0;
   if (H <= 0 || H > 65535 || !(cap > 0.f)) return QB_ERR_BAD_ARG;
-  const int threads = T <= R * DS_GATE_RUN ? 32 : 256;
+  if (T == R) {                                     // every request of a step brings at least one token
+    memory_gates_single_kernel<<<(R * H + 63) / 64, 64, 0, stream>>>(proj, stride, i_off, f_off, i_bias, f_bias, cap, m_state,
+                                                                     log_decay, weight, floor_out, req_slot, R, H);
+    QB_LAUNCH_CHECK();
+    return 0;
+  }
+  int threads = 64;
+  while (threads < 1024 && threads * DS_GATE_RUN < T) threads *= 2;
   memory_gates_kernel<<<dim3(R, H), threads, 0, stream>>>(proj, stride, i_off, f_off, i_bias, f_bias, cap, m_state,
                                                          log_decay, weight, floor_out, req_start, req_slot, H);
   QB_LAUNCH_CHECK();
@@ -151,7 +178,7 @@ extern "C" int qb_memory_gates(const float* proj, int stride, int i_off, int f_o
 // ---------------------------------------------------------------------------------------------
 // token by token, float32
 // ---------------------------------------------------------------------------------------------
-constexpr int DS_TB = 4;               // tokens a turn
+constexpr int DS_TURN = 4;             // tokens a turn (one where every request brings a single token)
 constexpr int DS_CHAIN_THREADS = 256;
 
 struct DsShape {
@@ -159,21 +186,21 @@ struct DsShape {
   long long stride;                    // elements between two token rows of q, k and v
 };
 
-// VEC columns a thread (4, or 1 where E is no multiple of 4), NR rows a thread; cols: columns a block.
-template <typename U, int VEC, int NR>
-__global__ void __launch_bounds__(DS_CHAIN_THREADS)
+// VEC columns a thread (4, or 1 where E is no multiple of 4), NR rows a thread, TB tokens a turn; cols: columns a block.
+template <typename U, int VEC, int NR, int TB>
+__global__ void __launch_bounds__(DS_CHAIN_THREADS, TB == 1 && VEC == 4 && NR <= 4 ? 4 : 1)
 ds_chain_kernel(const U* __restrict__ q, const U* __restrict__ k, const U* __restrict__ v, DsShape sh, DsGates gates,
                 float* __restrict__ state, float* __restrict__ n_state, const float* __restrict__ floor_in,
                 float* __restrict__ den, float* __restrict__ out, const int* __restrict__ req_start,
                 const int* __restrict__ req_slot, float q_scale, int silu, int cols, int max_tokens) {
   extern __shared__ __align__(16) float ds_sm[];
   const int D = sh.D, E = sh.E, H = sh.H;
-  float* s_k = ds_sm;                          // [DS_TB][D]
-  float* s_q = s_k + DS_TB * D;                // [DS_TB][D]
-  float* s_v = s_q + DS_TB * D;                // [DS_TB][cols]
-  float* s_red = s_v + DS_TB * cols;           // [warps][DS_TB][cols]
-  float* s_a = s_red + (DS_CHAIN_THREADS / 32) * DS_TB * cols;   // [DS_TB]
-  float* s_w = s_a + DS_TB;                    // [DS_TB]
+  float* s_k = ds_sm;                          // [TB][D]
+  float* s_q = s_k + TB * D;                // [TB][D]
+  float* s_v = s_q + TB * D;                // [TB][cols]
+  float* s_red = s_v + TB * cols;           // [warps][TB][cols]
+  float* s_a = s_red + (DS_CHAIN_THREADS / 32) * TB * cols;   // [TB]
+  float* s_w = s_a + TB;                    // [TB]
   const int r = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * cols;
   const int t0 = req_start[r], t1 = req_start[r + 1];
   if (t1 <= t0 || t1 - t0 > max_tokens) return;
@@ -208,8 +235,8 @@ ds_chain_kernel(const U* __restrict__ q, const U* __restrict__ k, const U* __res
   for (int u = 0; u < 8; ++u) nn[u] = norms && lane + 32 * u < D ? N[lane + 32 * u] : 0.f;
 
   auto act = [&](float x) { return silu ? x / (1.f + expf(-x)) : x; };
-  for (int tb = t0; tb < t1; tb += DS_TB) {
-    const int nt = min(DS_TB, t1 - tb);
+  for (int tb = t0; tb < t1; tb += TB) {
+    const int nt = min(TB, t1 - tb);
     for (int i = tid; i < nt * D; i += DS_CHAIN_THREADS) {
       const int tt = i / D, d = i % D;
       const size_t row = (size_t)(tb + tt) * sh.stride + (size_t)g * D + d;
@@ -227,9 +254,9 @@ ds_chain_kernel(const U* __restrict__ q, const U* __restrict__ k, const U* __res
       s_w[tid] = w;
     }
     __syncthreads();
-    float acc[DS_TB][VEC];
+    float acc[TB][VEC];
 #pragma unroll
-    for (int tt = 0; tt < DS_TB; ++tt) {
+    for (int tt = 0; tt < TB; ++tt) {
 #pragma unroll
       for (int c = 0; c < VEC; ++c) acc[tt][c] = 0.f;
       if (tt < nt) {
@@ -272,12 +299,14 @@ ds_chain_kernel(const U* __restrict__ q, const U* __restrict__ k, const U* __res
     }
     // the row groups' sums: lanes of the same columns, then the warps in order
 #pragma unroll
-    for (int tt = 0; tt < DS_TB; ++tt) {
+    for (int tt = 0; tt < TB; ++tt) {
 #pragma unroll
       for (int c = 0; c < VEC; ++c) {
-        float x = acc[tt][c];
-        for (int o = CQ; o < 32; o <<= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
-        if (lane < CQ) s_red[(warp * DS_TB + tt) * cols + cq * VEC + c] = x;
+        if (tt < nt) {
+          float x = acc[tt][c];
+          for (int o = CQ; o < 32; o <<= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+          if (lane < CQ) s_red[(warp * TB + tt) * cols + cq * VEC + c] = x;
+        }
       }
     }
     __syncthreads();
@@ -286,7 +315,7 @@ ds_chain_kernel(const U* __restrict__ q, const U* __restrict__ k, const U* __res
       if (e0 + c < E) {
         float x = 0.f;
 #pragma unroll
-        for (int w = 0; w < DS_CHAIN_THREADS / 32; ++w) x += s_red[(w * DS_TB + tt) * cols + c];
+        for (int w = 0; w < DS_CHAIN_THREADS / 32; ++w) x += s_red[(w * TB + tt) * cols + c];
         out[((size_t)(tb + tt) * H + h) * E + e0 + c] = x * q_scale;
       }
     }
@@ -324,27 +353,32 @@ extern "C" int qb_decay_chain(const void* q, const void* k, const void* v, int i
   const int rg = DS_CHAIN_THREADS / (cols / (vec ? 4 : 1));
   const int nr = (D + rg - 1) / rg;
   const dim3 grid(R, H, (E + cols - 1) / cols);
-  const size_t smem = (size_t)(DS_TB * (2 * D + cols) + (DS_CHAIN_THREADS / 32) * DS_TB * cols + 2 * DS_TB) * sizeof(float);
+  const bool single = T == R;                       // every request of a step brings at least one token
+  const int turn = single ? 1 : DS_TURN;
+  const size_t smem = (size_t)turn * (2 * D + cols + (DS_CHAIN_THREADS / 32) * cols + 2) * sizeof(float);
   const DsShape sh{H, G, D, E, stride};
   const DsGates gates{kind, decay, log_decay, step, step_stride, step_bias, A_log, weight};
 #define DS_CHAIN(VEC, NR)                                                                                          \
-  ds_chain_kernel<U, VEC, NR><<<grid, DS_CHAIN_THREADS, smem, stream>>>(                                           \
+  if (single) DS_CHAIN_TURN(VEC, NR, 1); else DS_CHAIN_TURN(VEC, NR, DS_TURN)
+#define DS_CHAIN_TURN(VEC, NR, TB_)                                                                                \
+  ds_chain_kernel<U, VEC, NR, TB_><<<grid, DS_CHAIN_THREADS, smem, stream>>>(                                           \
       (const U*)q, (const U*)k, (const U*)v, sh, gates, state, n_state, floor_in, den, out, req_start, req_slot,   \
       q_scale, silu, cols, max_tokens)
   QB_DISPATCH_DTYPE(in_dtype, U, {
     if (vec) {
-      if (nr <= 1) DS_CHAIN(4, 1);
-      else if (nr <= 2) DS_CHAIN(4, 2);
-      else if (nr <= 4) DS_CHAIN(4, 4);
-      else DS_CHAIN(4, 8);
+      if (nr <= 1) { DS_CHAIN(4, 1); }
+      else if (nr <= 2) { DS_CHAIN(4, 2); }
+      else if (nr <= 4) { DS_CHAIN(4, 4); }
+      else { DS_CHAIN(4, 8); }
     } else {
-      if (nr <= 4) DS_CHAIN(1, 4);
-      else if (nr <= 8) DS_CHAIN(1, 8);
-      else if (nr <= 16) DS_CHAIN(1, 16);
-      else DS_CHAIN(1, 32);
+      if (nr <= 4) { DS_CHAIN(1, 4); }
+      else if (nr <= 8) { DS_CHAIN(1, 8); }
+      else if (nr <= 16) { DS_CHAIN(1, 16); }
+      else { DS_CHAIN(1, 32); }
     }
   });
 #undef DS_CHAIN
+#undef DS_CHAIN_TURN
   QB_LAUNCH_CHECK();
   return 0;
 }

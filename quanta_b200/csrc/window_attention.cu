@@ -606,6 +606,13 @@ __device__ __forceinline__ float wm_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// cap * tanh(x / cap) as cap - 2 cap / (2^(x * two_over) + 1), two_over = 2 log2(e) / cap: two approximate instructions, whose
+// error is that of a float32 next to cap; the ends saturate at +-cap
+__device__ __forceinline__ float wm_cap(float x, float cap, float two_over) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(wm_exp2(x * two_over) + 1.f));
+  return fmaf(-2.f * cap, r, cap);
+}
 // two floats -> their bfloat16 roundings (hi) and the roundings of what is left (lo), each packed low | high
 __device__ __forceinline__ void wm_split_pair(float x, float y, uint32_t& hi, uint32_t& lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
@@ -665,6 +672,7 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
   // scores are kept times log2(e), so that a weight is one 2^x
   constexpr float LOG2E = 1.4426950408889634f;
   const bool plain = !(P.cap > 0.f) && P.dist_bias == nullptr;
+  const float two_over = P.cap > 0.f ? 2.f * LOG2E / P.cap : 0.f;
   const float mul = plain ? P.scale * LOG2E : P.scale;
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
   float o[NTV][4];
@@ -792,7 +800,7 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float x = s[nt][e] * mul;
-            if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
+            if (P.cap > 0.f) x = wm_cap(x, P.cap, two_over);
             if (P.dist_bias != nullptr) x += (e >= 2 ? bias_b : bias_a)[-(nt * 8 + (e & 1))];
             if (!plain) x *= LOG2E;
             s[nt][e] = x;
@@ -813,14 +821,14 @@ window_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bflo
             if (idx < nb_max) {
               if (idx < (second ? nb_b : nb_a)) {
                 x = s[nt][e] * mul;
-                if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
+                if (P.cap > 0.f) x = wm_cap(x, P.cap, two_over);
                 if (!plain) x *= LOG2E;
               }
             } else {
               const int j = lo_min + (idx - nb_max);
               if (j >= (second ? lo_b : lo_a) && j <= pos) {
                 x = s[nt][e] * mul;
-                if (P.cap > 0.f) x = P.cap * tanhf(x / P.cap);
+                if (P.cap > 0.f) x = wm_cap(x, P.cap, two_over);
                 if (P.dist_bias != nullptr) {
                   const int dd = pos - j - d0;
                   x += (dd >= 0 && dd < 2 * WM_BN) ? s_bias[dd] : __ldg(P.dist_bias + (size_t)(pos - j) * nq + h);

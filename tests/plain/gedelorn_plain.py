@@ -170,14 +170,17 @@ def squared_expert(w, p: str, h):
     return (F.relu(h @ w[p + "up"].T) ** 2) @ w[p + "down"].T
 
 
-def routed_ff(w, p: str, h, m: dict):
-    """The ``top`` largest of the sigmoid scores; their weights are the scores divided by their sum, times ``scale``;
-    a shared expert is added.  Returns (output, chosen [T, top], margin [T]: last chosen over first not chosen)."""
+def routed_ff(w, p: str, h, m: dict, chosen=None):
+    """The ``top`` largest of the sigmoid scores (or the experts ``chosen`` [T, top]); their weights are the scores divided
+    by their sum, times ``scale``; a shared expert is added.  Returns (output, chosen [T, top], margin [T]: last chosen over first not chosen)."""
     E, top, scale = int(m["router"]["experts"]), int(m["router"]["top"]), float(m["router"]["scale"])
     s = torch.sigmoid(h @ w[p + "router"].T)
     order = torch.sort(s, dim=-1, descending=True, stable=True)
     idx, val = order.indices[:, :top], order.values[:, :top]
     margin = val[:, -1] - order.values[:, top] if E > top else torch.full_like(s[:, 0], 1e9)
+    if chosen is not None:
+        idx = chosen.long()
+        val = s.gather(1, idx)
     weight = val / (val.sum(-1, keepdim=True) + 1e-20) * scale
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
@@ -190,15 +193,16 @@ def routed_ff(w, p: str, h, m: dict):
 
 # ---- the whole model -----------------------------------------------------------------------------------------
 def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: bool = False, disturb=None,
-            margins: list | None = None):
+            margins: list | None = None, chosen=None):
     """Logits ``[T, vocab]`` of one whole sequence; ``details``: also the stream after every layer; ``disturb``: applied
-    to what every sublayer reads (to see how much a model makes of a rounding); ``margins`` receives the routers'."""
+    to what every sublayer reads (to see how much a model makes of a rounding); ``margins`` receives the routers'; ``chosen``: per
+    routed layer, experts [T, top] to take instead of choosing."""
     seen = disturb or (lambda t: t)
     w = {k: (v.to(dtype) if v.is_floating_point() else v) for k, v in weights.items()}
     eps = float(config["norm"]["eps"])
     ids = torch.as_tensor(tokens, dtype=torch.long, device=w["embed"].device)
     x = w["embed"][ids]
-    after = []
+    after, routed = [], 0
     for i, layer in enumerate(config["layers"]):
         p, m = f"l{i}.", layer["mixer"]
         h = seen(around_zero_norm(x, w[p + "norm1"], eps))
@@ -217,7 +221,8 @@ def forward(weights: dict, config: dict, tokens, dtype=torch.float32, details: b
             if mlp["kind"] == "dense":
                 y = gated_ff(w, p + "mlp.", h)
             else:
-                y, _, margin = routed_ff(w, p + "mlp.", h, mlp)
+                y, _, margin = routed_ff(w, p + "mlp.", h, mlp, None if chosen is None else chosen[routed])
+                routed += 1
                 if margins is not None:
                     margins.append(margin)
             x = x + around_zero_norm(y, w[p + "norm2b"], eps)

@@ -35,7 +35,8 @@ UNITS = {
     "rope": ["rope_cache.cu"],
     "attention": ["attention_simt.cu", "attention_mma.cu", "attention_tc.cu"],
     "experts": ["moe.cu", "router_gemm_mma.cu", "expert_gemm_tc.cu"],
-    "recurrent": ["short_conv.cu", "delta_rule.cu", "gated_delta.cu"],
+    "short_conv": ["short_conv.cu"],
+    "recurrent": ["delta_rule.cu", "gated_delta.cu"],
     "latent": ["latent_attention.cu"],
     "linear_attention": ["gla.cu"],
     "window_attention": ["window_attention.cu"],

@@ -387,6 +387,7 @@ extern "C" int qb_decay_chain(const void* q, const void* k, const void* v, int i
 // chunks of tokens on the tensor cores
 // ---------------------------------------------------------------------------------------------
 constexpr int DS_C = 64;                // tokens a chunk
+constexpr int DS_CHUNK_THREADS = 256;
 constexpr int DS_DIRECT = 0, DS_LOCAL = 1, DS_REPLAY = 2;
 
 __device__ __forceinline__ void ds_ldsm(uint32_t (&r)[4], const void* p) {
@@ -480,16 +481,19 @@ __global__ void ds_combine_kernel(float* __restrict__ state, float* __restrict__
   }
 }
 
-// NM: 16-row tiles of S a warp holds (four warps; D <= 64 NM); ET: columns a block; LOCAL: no outputs, from a zero state.
+// NM: D <= 64 NM; ET: columns a block; LOCAL: no outputs, from a zero state.  Eight warps: of the outputs a warp takes 16
+// tokens and half of the columns (both halves of a token work out its scores); of S it takes MT tiles of 16 channels and
+// SN of the NT tiles of 8 columns.
 template <int NM, int ET, bool LOCAL>
-__global__ void __launch_bounds__(128, NM <= 2 ? 2 : 1)
+__global__ void __launch_bounds__(DS_CHUNK_THREADS, NM <= 2 ? 2 : 1)
 ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k,
                 const __nv_bfloat16* __restrict__ v, DsShape sh, DsGates gates, float* __restrict__ state,
                 float* __restrict__ n_state, const float* __restrict__ floor_in, float* __restrict__ den,
                 float* __restrict__ out, const int* __restrict__ req_start, const int* __restrict__ req_slot,
                 const int4* __restrict__ seg, const int* __restrict__ n_seg, float* __restrict__ seg_state,
                 float* __restrict__ seg_n, float* __restrict__ seg_log, int mode, float q_scale, int min_tokens) {
-  constexpr int DP = 64 * NM, PK = DP + 8, PV = ET + 8, NT = ET / 8;
+  constexpr int DP = 64 * NM, PK = DP + 8, PV = ET + 8, NT = ET / 8, NO = NT / 2;
+  constexpr int MT = NM == 4 ? 2 : 1, SN = NM == 1 ? NT / 2 : NT;
   extern __shared__ __align__(16) unsigned char ds_raw[];
   __nv_bfloat16* Ks0 = reinterpret_cast<__nv_bfloat16*>(ds_raw);       // [2][64][PK]
   __nv_bfloat16* Vs0 = Ks0 + 2 * DS_C * PK;                            // [2][64][PV]
@@ -506,6 +510,9 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
   const int D = sh.D, E = sh.E, H = sh.H;
   const int h = blockIdx.y, e0 = blockIdx.z * ET;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+  const int tw = warp & 3, o_tile = (warp >> 2) * NO;                 // token tile and first column tile of the outputs
+  const int s_tile = NM == 1 ? (warp >> 2) * SN : 0;                   // first column tile of S
+  auto s_chan = [&](int u) { return (NM == 1 ? tw : 8 * u + warp) * 16; };   // first channel of S tile u
   int t0, t1;
   float *S, *N = nullptr;
   const bool norms = n_state != nullptr && blockIdx.z == 0;
@@ -531,20 +538,19 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
   const int dc = D / 8, ec = min(ET, E - e0) / 8;                      // 16-byte pieces a row
 
   // what no copy ever writes (channels past D, columns past E, rows past a last chunk's end) is read as zeros
-  for (int i = tid; i < (2 * DS_C * (PK + PV)) / 8; i += 128) reinterpret_cast<uint4*>(Ks0)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < (2 * DS_C * (PK + PV)) / 8; i += DS_CHUNK_THREADS) reinterpret_cast<uint4*>(Ks0)[i] = make_uint4(0, 0, 0, 0);
   if (!LOCAL)
-    for (int i = tid; i < DS_C * PK / 8; i += 128) reinterpret_cast<uint4*>(Qs)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < DP; i += 128) s_n[i] = (norms && !LOCAL && i < D) ? N[i] : 0.f;
+    for (int i = tid; i < DS_C * PK / 8; i += DS_CHUNK_THREADS) reinterpret_cast<uint4*>(Qs)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < DP; i += DS_CHUNK_THREADS) s_n[i] = (norms && !LOCAL && i < D) ? N[i] : 0.f;
 
-  // this warp's rows of S: tile u covers the channels (4 u + warp) * 16 ..
-  float s[NM][NT][4];
+  float s[MT][SN][4];
 #pragma unroll
-  for (int u = 0; u < NM; ++u)
+  for (int u = 0; u < MT; ++u)
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int n = 0; n < SN; ++n)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const int d = (4 * u + warp) * 16 + g8 + 8 * half, e = e0 + n * 8 + 2 * t4;
+        const int d = s_chan(u) + g8 + 8 * half, e = e0 + (s_tile + n) * 8 + 2 * t4;
         float2 x = make_float2(0.f, 0.f);
         if (!LOCAL && d < D && e < E) x = *reinterpret_cast<const float2*>(S + (size_t)d * E + e);
         s[u][n][2 * half] = x.x;
@@ -554,7 +560,7 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
 
   auto copy = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int pieces, int c0) {
     const int n = min(DS_C, t1 - c0) * pieces;
-    for (int i = tid; i < n; i += 128) {
+    for (int i = tid; i < n; i += DS_CHUNK_THREADS) {
       const int tt = i / pieces, c = i % pieces;
       const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst + tt * pitch + c * 8);
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(to), "l"(src + (size_t)(c0 + tt) * sh.stride + c * 8) : "memory");
@@ -609,14 +615,14 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
     if (!LOCAL) {
       // S as it stands before the chunk, in two parts
 #pragma unroll
-      for (int u = 0; u < NM; ++u)
+      for (int u = 0; u < MT; ++u)
 #pragma unroll
-        for (int n = 0; n < NT; ++n)
+        for (int n = 0; n < SN; ++n)
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
             uint32_t hi, lo;
             ds_split(s[u][n][2 * half], s[u][n][2 * half + 1], hi, lo);
-            const int at = ((4 * u + warp) * 16 + g8 + 8 * half) * PV + n * 8 + 2 * t4;
+            const int at = (s_chan(u) + g8 + 8 * half) * PV + (s_tile + n) * 8 + 2 * t4;
             *reinterpret_cast<uint32_t*>(Sh + at) = hi;
             *reinterpret_cast<uint32_t*>(Sl + at) = lo;
           }
@@ -629,18 +635,18 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       asm volatile("cp.async.commit_group;\n" ::: "memory");
     }
     if (!LOCAL) {
-      const int ra = warp * 16 + g8, rb = ra + 8;                      // this thread's two tokens
+      const int ra = tw * 16 + g8, rb = ra + 8;                      // this thread's two tokens
       const float hi_a = s_hi[ra], hi_b = s_hi[rb], lo_a = s_lo[ra], lo_b = s_lo[rb];
-      float o[NT][4];
+      float o[NO][4];
 #pragma unroll
-      for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+      for (int n = 0; n < NO; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
       for (int kk = 0; kk < kd; ++kk) {
         uint32_t a[4];
-        ds_ldsm(a, Qs + (warp * 16 + lane % 16) * PK + kk * 16 + (lane / 16) * 8);
+        ds_ldsm(a, Qs + (tw * 16 + lane % 16) * PK + kk * 16 + (lane / 16) * 8);
 #pragma unroll
-        for (int n = 0; n < NT; n += 2) {
+        for (int n = 0; n < NO; n += 2) {
           uint32_t b[4];
-          const int at = (kk * 16 + lane % 16) * PV + n * 8 + (lane / 16) * 8;
+          const int at = (kk * 16 + lane % 16) * PV + (o_tile + n) * 8 + (lane / 16) * 8;
           ds_ldsm_t(b, Sh + at);
           ds_mma(o[n], a, b[0], b[1]);
           ds_mma(o[n + 1], a, b[2], b[3]);
@@ -651,16 +657,16 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       }
       const float el_a = ds_exp2(hi_a + lo_a), el_b = ds_exp2(hi_b + lo_b);
 #pragma unroll
-      for (int n = 0; n < NT; ++n) {
+      for (int n = 0; n < NO; ++n) {
         o[n][0] *= el_a; o[n][1] *= el_a;
         o[n][2] *= el_b; o[n][3] *= el_b;
       }
       float sum_a = 0.f, sum_b = 0.f;
-      for (int kt = 0; kt <= warp && kt * 16 < nt; ++kt) {             // keys of 16 tokens a turn, none after the rows'
+      for (int kt = 0; kt <= tw && kt * 16 < nt; ++kt) {             // keys of 16 tokens a turn, none after the rows'
         float p[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
         for (int kk = 0; kk < kd; ++kk) {
           uint32_t a[4], b[4];
-          ds_ldsm(a, Qs + (warp * 16 + lane % 16) * PK + kk * 16 + (lane / 16) * 8);
+          ds_ldsm(a, Qs + (tw * 16 + lane % 16) * PK + kk * 16 + (lane / 16) * 8);
           ds_ldsm(b, Ks + (kt * 16 + (lane / 16) * 8 + lane % 8) * PK + kk * 16 + ((lane / 8) % 2) * 8);
           ds_mma(p[0], a, b[0], b[1]);
           ds_mma(p[1], a, b[2], b[3]);
@@ -682,9 +688,9 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
         ds_split(p[1][0], p[1][1], ph[2], pl[2]);
         ds_split(p[1][2], p[1][3], ph[3], pl[3]);
 #pragma unroll
-        for (int n = 0; n < NT; n += 2) {
+        for (int n = 0; n < NO; n += 2) {
           uint32_t b[4];
-          ds_ldsm_t(b, Vs + (kt * 16 + lane % 16) * PV + n * 8 + (lane / 16) * 8);
+          ds_ldsm_t(b, Vs + (kt * 16 + lane % 16) * PV + (o_tile + n) * 8 + (lane / 16) * 8);
           ds_mma(o[n], ph, b[0], b[1]);
           ds_mma(o[n + 1], ph, b[2], b[3]);
           ds_mma(o[n], pl, b[0], b[1]);
@@ -692,14 +698,14 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
         }
       }
 #pragma unroll
-      for (int n = 0; n < NT; ++n) {
-        const int e = e0 + n * 8 + 2 * t4;
+      for (int n = 0; n < NO; ++n) {
+        const int e = e0 + (o_tile + n) * 8 + 2 * t4;
         if (e < E) {
           if (ra < nt) *reinterpret_cast<float2*>(out + ((size_t)(c0 + ra) * H + h) * E + e) = make_float2(o[n][0] * q_scale, o[n][1] * q_scale);
           if (rb < nt) *reinterpret_cast<float2*>(out + ((size_t)(c0 + rb) * H + h) * E + e) = make_float2(o[n][2] * q_scale, o[n][3] * q_scale);
         }
       }
-      if (norms) {
+      if (norms && warp < 4) {
         // n . q = the row sum of the weighted scores + the decayed old n . q: two threads a token
         sum_a += __shfl_xor_sync(0xffffffffu, sum_a, 1);
         sum_a += __shfl_xor_sync(0xffffffffu, sum_a, 2);
@@ -724,7 +730,7 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       }
     }
     // values weighted to the chunk's end, in two parts
-    for (int i = tid; i < DS_C * ET / 2; i += 128) {
+    for (int i = tid; i < DS_C * ET / 2; i += DS_CHUNK_THREADS) {
       const int tt = i / (ET / 2), c = (i % (ET / 2)) * 2;
       const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(Vs + tt * PV + c);
       const float w = s_wt[tt];
@@ -735,7 +741,7 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
     }
     const float keep = ds_exp2(s_tot[0]);
     if (norms) {
-      for (int d = tid; d < D; d += 128) {
+      for (int d = tid; d < D; d += DS_CHUNK_THREADS) {
         float x = s_n[d] * keep;
         for (int tt = 0; tt < nt; ++tt) x = fmaf(s_wt[tt], __bfloat162float(Ks[tt * PK + d]), x);
         s_n[d] = x;
@@ -743,27 +749,27 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
     }
     __syncthreads();
 #pragma unroll
-    for (int u = 0; u < NM; ++u)
+    for (int u = 0; u < MT; ++u)
 #pragma unroll
-      for (int n = 0; n < NT; ++n)
+      for (int n = 0; n < SN; ++n)
 #pragma unroll
         for (int c = 0; c < 4; ++c) s[u][n][c] *= keep;
 #pragma unroll
     for (int kt = 0; kt < DS_C / 16; ++kt) {
       if (kt * 16 < nt) {
-        uint32_t a[NM][4];
+        uint32_t a[MT][4];
 #pragma unroll
-        for (int u = 0; u < NM; ++u)
-          ds_ldsm_t(a[u], Ks + (kt * 16 + (lane / 16) * 8 + lane % 8) * PK + (4 * u + warp) * 16 + ((lane / 8) % 2) * 8);
+        for (int u = 0; u < MT; ++u)
+          ds_ldsm_t(a[u], Ks + (kt * 16 + (lane / 16) * 8 + lane % 8) * PK + s_chan(u) + ((lane / 8) % 2) * 8);
 #pragma unroll
-        for (int n = 0; n < NT; n += 2) {
+        for (int n = 0; n < SN; n += 2) {
           uint32_t bh[4], bl[4];
-          const int at = (kt * 16 + lane % 16) * PV + n * 8 + (lane / 16) * 8;
+          const int at = (kt * 16 + lane % 16) * PV + (s_tile + n) * 8 + (lane / 16) * 8;
           ds_ldsm_t(bh, Vs + at);
           ds_ldsm_t(bl, Sl + at);
 #pragma unroll
-          for (int u = 0; u < NM; ++u) {
-            if ((4 * u + warp) * 16 < D) {
+          for (int u = 0; u < MT; ++u) {
+            if (s_chan(u) < D) {
               ds_mma(s[u][n], a[u], bh[0], bh[1]);
               ds_mma(s[u][n + 1], a[u], bh[2], bh[3]);
               ds_mma(s[u][n], a[u], bl[0], bl[1]);
@@ -777,16 +783,16 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
   }
   if (mode != DS_REPLAY) {
 #pragma unroll
-    for (int u = 0; u < NM; ++u)
+    for (int u = 0; u < MT; ++u)
 #pragma unroll
-      for (int n = 0; n < NT; ++n)
+      for (int n = 0; n < SN; ++n)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int d = (4 * u + warp) * 16 + g8 + 8 * half, e = e0 + n * 8 + 2 * t4;
+          const int d = s_chan(u) + g8 + 8 * half, e = e0 + (s_tile + n) * 8 + 2 * t4;
           if (d < D && e < E) *reinterpret_cast<float2*>(S + (size_t)d * E + e) = make_float2(s[u][n][2 * half], s[u][n][2 * half + 1]);
         }
     if (norms)
-      for (int d = tid; d < D; d += 128) N[d] = s_n[d];
+      for (int d = tid; d < D; d += DS_CHUNK_THREADS) N[d] = s_n[d];
   }
   if (LOCAL && tid == 0 && blockIdx.z == 0) seg_log[(size_t)blockIdx.x * H + h] = (float)seg_total;
 }
@@ -852,7 +858,7 @@ extern "C" int qb_decay_chunks(const void* q, const void* k, const void* v, long
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
       if (e != cudaSuccess) return (int)e;                                                                               \
     }                                                                                                                    \
-    kern<<<dim3(GX, H, zt), 128, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, \
+    kern<<<dim3(GX, H, zt), DS_CHUNK_THREADS, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, \
         sh, gates, state, n_state, floor_in, den, out, req_start, req_slot, seg, n_seg, seg_state, seg_n, seg_log, MODE_, \
         q_scale, min_tokens);                                                                                            \
   } while (0)

@@ -481,6 +481,9 @@ __global__ void ds_combine_kernel(float* __restrict__ state, float* __restrict__
   }
 }
 
+struct DsTrue { static constexpr bool value = true; };
+struct DsFalse { static constexpr bool value = false; };
+
 // NM: D <= 64 NM; ET: columns a block; LOCAL: no outputs, from a zero state.  Eight warps: of the outputs a warp takes 16
 // tokens and half of the columns (both halves of a token work out its scores); of S it takes MT tiles of 16 channels and
 // SN of the NT tiles of 8 columns.
@@ -500,13 +503,12 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
   __nv_bfloat16* Sl = Vs0 + 2 * DS_C * PV;                             // [DP][PV]: the low parts of S, then of the weighted values
   __nv_bfloat16* Sh = Sl + (LOCAL ? DS_C : DP) * PV;                   // [DP][PV]
   __nv_bfloat16* Qs = Sh + (LOCAL ? 0 : DP) * PV;                      // [64][PK]
-  float* s_hi = reinterpret_cast<float*>(Qs + (LOCAL ? 0 : DS_C) * PK);  // [64] log2 of the cumulated decay, its two parts
-  float* s_lo = s_hi + DS_C;                                           // [64]
-  float* s_w = s_lo + DS_C;                                            // [64] weights
-  float* s_wt = s_w + DS_C;                                            // [64] weights decayed to the chunk's end
-  float* s_rs = s_wt + DS_C;                                           // [64] row sums of the weighted scores
+  // a chunk's gates, two buffers: log2 of the cumulated decay in two parts, weights, weights decayed to the end of their 16
+  // tokens, weights decayed to the chunk's end (64 of each), log2 of the chunk's decay
+  constexpr int GB = 5 * DS_C + 4;
+  float* s_gate = reinterpret_cast<float*>(Qs + (LOCAL ? 0 : DS_C) * PK);
+  float* s_rs = s_gate + 2 * GB;                                       // [64] row sums of the weighted scores
   float* s_n = s_rs + DS_C;                                            // [DP] the normaliser
-  float* s_tot = s_n + DP;                                             // [1] log2 of the chunk's decay
   const int D = sh.D, E = sh.E, H = sh.H;
   const int h = blockIdx.y, e0 = blockIdx.z * ET;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
@@ -558,60 +560,75 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       }
   __syncthreads();
 
-  auto copy = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int pieces, int c0) {
-    const int n = min(DS_C, t1 - c0) * pieces;
-    for (int i = tid; i < n; i += DS_CHUNK_THREADS) {
-      const int tt = i / pieces, c = i % pieces;
-      const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst + tt * pitch + c * 8);
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(to), "l"(src + (size_t)(c0 + tt) * sh.stride + c * 8) : "memory");
+  // rows of q, k (KEYS) or v of the chunk at c0 by asynchronous copies of 16 bytes; a thread keeps its column
+  auto copy = [&](auto keys, __nv_bfloat16* dst, const __nv_bfloat16* src, int pieces, int c0) {
+    constexpr bool KEYS = decltype(keys)::value;
+    constexpr int SLOTS = KEYS ? DP / 8 : ET / 8, pitch = KEYS ? PK : PV;
+    const int c = tid % SLOTS, nt = min(DS_C, t1 - c0);
+    if (c < pieces) {
+#pragma unroll
+      for (int tt = tid / SLOTS; tt < DS_C; tt += DS_CHUNK_THREADS / SLOTS) {
+        if (tt < nt) {
+          const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst + tt * pitch + c * 8);
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(to), "l"(src + (size_t)(c0 + tt) * sh.stride + c * 8) : "memory");
+        }
+      }
     }
   };
+  constexpr DsTrue of_keys{};
+  constexpr DsFalse of_values{};
   const __nv_bfloat16* k_src = k + (size_t)g * D;
   const __nv_bfloat16* q_src = q + (size_t)g * D;
   const __nv_bfloat16* v_src = v + (size_t)h * E + e0;
-  copy(Ks0, PK, k_src, dc, t0);
-  copy(Vs0, PV, v_src, ec, t0);
-  if (!LOCAL) copy(Qs, PK, q_src, dc, t0);
+  copy(of_keys, Ks0, k_src, dc, t0);
+  copy(of_values, Vs0, v_src, ec, t0);
+  if (!LOCAL) copy(of_keys, Qs, q_src, dc, t0);
   asm volatile("cp.async.commit_group;\n" ::: "memory");
 
   double seg_total = 0.0;                 // warp 0: log2 of the segment's decay so far
+  // warp 0, two tokens a lane: the gates of the chunk at c0, cumulated over the chunk
+  auto gates_of = [&](int c0, float* s_hi) {
+    const int nt = min(DS_C, t1 - c0);
+    float *s_lo = s_hi + DS_C, *s_w = s_lo + DS_C, *s_wl = s_w + DS_C, *s_wt = s_wl + DS_C;
+    float la[2] = {0.f, 0.f}, w[2] = {0.f, 0.f};
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+      if (2 * lane + u < nt) {
+        ds_log_gate(gates, c0 + 2 * lane + u, h, H, la[u], w[u]);
+        la[u] = fmaxf(la[u], DS_LOG_FLOOR);
+      }
+    const double LOG2E = 1.4426950408889634;
+    const double x0 = (double)la[0] * LOG2E, x1 = x0 + (double)la[1] * LOG2E;
+    double sum = x1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const double p = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += p;
+    }
+    const double total = __shfl_sync(0xffffffffu, sum, 31);
+    const double tile_end = __shfl_sync(0xffffffffu, sum, lane | 7);   // eight lanes hold 16 tokens
+    const double before = sum - x1;
+    const double L[2] = {before + x0, sum};
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = 2 * lane + u;
+      s_hi[i] = (float)L[u];
+      s_lo[i] = (float)(L[u] - (double)(float)L[u]);
+      s_w[i] = w[u];
+      s_wl[i] = ds_exp2((float)(tile_end - L[u])) * w[u];
+      s_wt[i] = ds_exp2((float)(total - L[u])) * w[u];
+    }
+    if (lane == 0) s_wt[DS_C] = (float)total;
+    seg_total += total;
+  };
+  if (warp == 0) gates_of(t0, s_gate);
   int buf = 0;
   for (int c0 = t0; c0 < t1; c0 += DS_C, buf ^= 1) {
     const int nt = min(DS_C, t1 - c0);
     const bool more = c0 + DS_C < t1;
     __nv_bfloat16* Ks = Ks0 + buf * DS_C * PK;
     __nv_bfloat16* Vs = Vs0 + buf * DS_C * PV;
-    if (warp == 0) {
-      // two tokens a lane: their gates, cumulated over the chunk
-      float la[2] = {0.f, 0.f}, w[2] = {0.f, 0.f};
-#pragma unroll
-      for (int u = 0; u < 2; ++u)
-        if (2 * lane + u < nt) {
-          ds_log_gate(gates, c0 + 2 * lane + u, h, H, la[u], w[u]);
-          la[u] = fmaxf(la[u], DS_LOG_FLOOR);
-        }
-      const double LOG2E = 1.4426950408889634;
-      const double x0 = (double)la[0] * LOG2E, x1 = x0 + (double)la[1] * LOG2E;
-      double sum = x1;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const double p = __shfl_up_sync(0xffffffffu, sum, o);
-        if (lane >= o) sum += p;
-      }
-      const double total = __shfl_sync(0xffffffffu, sum, 31);
-      const double before = sum - x1;
-      const double L[2] = {before + x0, before + x1};
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int i = 2 * lane + u;
-        s_hi[i] = (float)L[u];
-        s_lo[i] = (float)(L[u] - (double)(float)L[u]);
-        s_w[i] = w[u];
-        s_wt[i] = ds_exp2((float)(total - L[u])) * w[u];
-      }
-      if (lane == 0) s_tot[0] = (float)total;
-      seg_total += total;
-    }
+    const float *s_hi = s_gate + buf * GB, *s_lo = s_hi + DS_C, *s_w = s_lo + DS_C, *s_wl = s_w + DS_C, *s_wt = s_wl + DS_C;
     if (!LOCAL) {
       // S as it stands before the chunk, in two parts
 #pragma unroll
@@ -630,9 +647,10 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
     __syncthreads();
     if (more) {
-      copy(Ks0 + (buf ^ 1) * DS_C * PK, PK, k_src, dc, c0 + DS_C);
-      copy(Vs0 + (buf ^ 1) * DS_C * PV, PV, v_src, ec, c0 + DS_C);
+      copy(of_keys, Ks0 + (buf ^ 1) * DS_C * PK, k_src, dc, c0 + DS_C);
+      copy(of_values, Vs0 + (buf ^ 1) * DS_C * PV, v_src, ec, c0 + DS_C);
       asm volatile("cp.async.commit_group;\n" ::: "memory");
+      if (warp == 0) gates_of(c0 + DS_C, s_gate + (buf ^ 1) * GB);     // its tokens have the fewest keys in this chunk
     }
     if (!LOCAL) {
       const int ra = tw * 16 + g8, rb = ra + 8;                      // this thread's two tokens
@@ -671,17 +689,34 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
           ds_mma(p[0], a, b[0], b[1]);
           ds_mma(p[1], a, b[2], b[3]);
         }
+        if (kt < tw) {
+          // all of these keys come before all of the warp's tokens: decays to the keys' last token, then on to the tokens
+          const float he = s_hi[kt * 16 + 15], le = s_lo[kt * 16 + 15];
+          const float f_a = ds_exp2((hi_a - he) + (lo_a - le)), f_b = ds_exp2((hi_b - he) + (lo_b - le));
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int c = 0; c < 2; ++c) {
-            const int j = kt * 16 + n * 8 + 2 * t4 + c;
-            const float hj = s_hi[j], lj = s_lo[j], wj = s_w[j];
-            p[n][c] = j <= ra ? p[n][c] * (ds_exp2((hi_a - hj) + (lo_a - lj)) * wj) : 0.f;
-            p[n][2 + c] = j <= rb ? p[n][2 + c] * (ds_exp2((hi_b - hj) + (lo_b - lj)) * wj) : 0.f;
-            sum_a += p[n][c];
-            sum_b += p[n][2 + c];
+          for (int n = 0; n < 2; ++n) {
+            const float2 w = *reinterpret_cast<const float2*>(s_wl + kt * 16 + n * 8 + 2 * t4);
+            p[n][0] *= f_a * w.x; p[n][1] *= f_a * w.y;
+            p[n][2] *= f_b * w.x; p[n][3] *= f_b * w.y;
           }
+        } else {
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+              const int j = kt * 16 + n * 8 + 2 * t4 + c;
+              const float hj = s_hi[j], lj = s_lo[j], wj = s_w[j];
+              p[n][c] = j <= ra ? p[n][c] * (ds_exp2((hi_a - hj) + (lo_a - lj)) * wj) : 0.f;
+              p[n][2 + c] = j <= rb ? p[n][2 + c] * (ds_exp2((hi_b - hj) + (lo_b - lj)) * wj) : 0.f;
+            }
+        }
+        if (norms) {
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            sum_a += p[n][0] + p[n][1];
+            sum_b += p[n][2] + p[n][3];
+          }
+        }
         uint32_t ph[4], pl[4];
         ds_split(p[0][0], p[0][1], ph[0], pl[0]);
         ds_split(p[0][2], p[0][3], ph[1], pl[1]);
@@ -725,7 +760,7 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       }
       __syncthreads();                    // Q, the unweighted values, the parts of S and n have been read
       if (more) {
-        copy(Qs, PK, q_src, dc, c0 + DS_C);
+        copy(of_keys, Qs, q_src, dc, c0 + DS_C);
         asm volatile("cp.async.commit_group;\n" ::: "memory");
       }
     }
@@ -739,7 +774,7 @@ ds_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __rest
       *reinterpret_cast<uint32_t*>(Vs + tt * PV + c) = hi;
       *reinterpret_cast<uint32_t*>(Sl + tt * PV + c) = lo;
     }
-    const float keep = ds_exp2(s_tot[0]);
+    const float keep = ds_exp2(s_wt[DS_C]);
     if (norms) {
       for (int d = tid; d < D; d += DS_CHUNK_THREADS) {
         float x = s_n[d] * keep;
@@ -852,7 +887,7 @@ extern "C" int qb_decay_chunks(const void* q, const void* k, const void* v, long
   do {                                                                                                                  \
     constexpr int DP = 64 * NM, PK = DP + 8, PV = ET + 8;                                                                \
     const size_t smem = (size_t)(2 * DS_C * (PK + PV) + (LOCAL_ ? DS_C * PV : 2 * DP * PV + DS_C * PK)) * 2 +            \
-                        (size_t)(5 * DS_C + DP + 4) * sizeof(float);                                                     \
+                        (size_t)(2 * (5 * DS_C + 4) + DS_C + DP) * sizeof(float);                                                     \
     auto kern = ds_chunk_kernel<NM, ET, LOCAL_>;                                                                         \
     if (smem > 48 * 1024) {                                                                                             \
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \

@@ -967,15 +967,16 @@ extern "C" int qb_rows_act(const float* x, long long stride, void* out, int out_
 //   y <- y * silu(gate)                                          (gate_first: the gate before the norm)
 //   y <- y / rms over each of `parts` equal parts of the row (eps inside the root) * gain
 //   y <- y * sigmoid(gate)                                       (else)
-// A group of threads a (token, part): a warp for parts of up to 512 numbers, a block for longer ones; the part stays
-// in shared memory between the two passes.  Sums in an order that depends on the sizes alone.
+// A group of threads a (token, part): a warp for parts of up to 512 numbers, a block for longer ones.  Parts that move in
+// 16-byte pieces and fit (Q pieces a thread) are held in registers, with all loads asked for before the first sum; other
+// parts stay in shared memory between the two passes.  Sums in an order that depends on the sizes alone.
 // ---------------------------------------------------------------------------------------------
-template <typename O, int WARPS>       // warps a part: 1 (four parts a block) or 8
+template <typename O, int WARPS, int Q>       // WARPS a part: 1 (four parts a block) or 8; Q 0: shared memory, any sizes
 __global__ void __launch_bounds__(WARPS == 1 ? 128 : 256)
 decay_out_kernel(const float* __restrict__ o, const float* __restrict__ den, const O* __restrict__ x, long long x_stride,
                  const float* __restrict__ skip, const float* __restrict__ gate, long long gate_stride,
                  const float* __restrict__ gain, O* __restrict__ out, int T, int H, int E, int parts, float eps,
-                 int gate_first, int vec) {
+                 int gate_first) {
   extern __shared__ __align__(16) float s_part[];
   __shared__ float s_sum[32];
   const int HE = H * E, n = HE / parts;
@@ -983,72 +984,88 @@ decay_out_kernel(const float* __restrict__ o, const float* __restrict__ den, con
   const long long unit = (long long)blockIdx.x * (WARPS == 1 ? 4 : 1) + group;
   if (unit >= (long long)T * parts) return;           // a whole warp (or block) leaves
   const int t = (int)(unit / parts), c0 = (int)(unit % parts) * n;
-  float* buf = s_part + group * n;
   const float* orow = o + (size_t)t * HE + c0;
   const float* grow = gate + (size_t)t * gate_stride + c0;
-  float ss = 0.f;
-  auto value = [&](int i, float ov, float gv, float xv) {
-    const int h = (c0 + i) / E;
-    float y = ov;
-    if (den != nullptr) y = y / den[(size_t)t * H + h];
-    if (skip != nullptr) y = fmaf(skip[h], xv, y);
-    if (gate_first) y *= gv / (1.f + expf(-gv));
-    return y;
+  const float* nrow = gain + c0;
+  const O* xrow = skip != nullptr ? x + (size_t)t * x_stride + c0 : nullptr;
+  O* to = out + (size_t)t * HE + c0;
+  auto root = [&](float ss) {
+    if (WARPS == 1) {
+      ss = qb_warp_sum(ss);
+      __syncwarp();
+    } else {
+      ss = qb_block_sum(ss, s_sum);
+    }
+    return 1.f / sqrtf(ss / (float)n + eps);
   };
-  if (vec) {
-    for (int i = me * 4; i < n; i += nth * 4) {
-      const float4 ov = *reinterpret_cast<const float4*>(orow + i);
-      float4 gv = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (gate_first) gv = *reinterpret_cast<const float4*>(grow + i);
-      float xv[4] = {0.f, 0.f, 0.f, 0.f};
-      if (skip != nullptr) {
+  if constexpr (Q > 0) {
+    float4 y[Q], gv[Q], gn[Q];
+    float dn[Q], sk[Q], xv[Q][4];
+    struct alignas(4 * sizeof(O)) Four { O v[4]; };
 #pragma unroll
-        for (int e = 0; e < 4; ++e) xv[e] = qb_to_float<O>(x[(size_t)t * x_stride + c0 + i + e]);
+    for (int u = 0; u < Q; ++u) {
+      const int i = (me + u * nth) * 4;
+      dn[u] = 1.f;
+      sk[u] = 0.f;
+      if (i < n) {
+        const int h = (c0 + i) / E;                   // four numbers of one head
+        y[u] = *reinterpret_cast<const float4*>(orow + i);
+        gv[u] = *reinterpret_cast<const float4*>(grow + i);
+        gn[u] = *reinterpret_cast<const float4*>(nrow + i);
+        if (den != nullptr) dn[u] = den[(size_t)t * H + h];
+        if (skip != nullptr) {
+          sk[u] = skip[h];
+          const Four f = *reinterpret_cast<const Four*>(xrow + i);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) xv[u][e] = qb_to_float<O>(f.v[e]);
+        }
+      } else {
+        y[u] = gv[u] = gn[u] = make_float4(0.f, 0.f, 0.f, 0.f);
       }
-      float4 y;
-      y.x = value(i, ov.x, gv.x, xv[0]);
-      y.y = value(i + 1, ov.y, gv.y, xv[1]);
-      y.z = value(i + 2, ov.z, gv.z, xv[2]);
-      y.w = value(i + 3, ov.w, gv.w, xv[3]);
-      ss += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
-      *reinterpret_cast<float4*>(buf + i) = y;
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+      float* yv = &y[u].x;
+      float* g = &gv[u].x;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (den != nullptr) yv[e] /= dn[u];
+        if (skip != nullptr && (me + u * nth) * 4 < n) yv[e] = fmaf(sk[u], xv[u][e], yv[e]);
+        const float sg = 1.f / (1.f + expf(-g[e]));
+        if (gate_first) yv[e] *= g[e] * sg;           // silu before the norm
+        g[e] = gate_first ? 1.f : sg;                 // what multiplies the normed number
+        ss += yv[e] * yv[e];
+      }
+    }
+    const float inv = root(ss);
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+      const int i = (me + u * nth) * 4;
+      if (i < n) {
+        Four four;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) four.v[e] = qb_from_float<O>((&y[u].x)[e] * inv * (&gn[u].x)[e] * (&gv[u].x)[e]);
+        *reinterpret_cast<Four*>(to + i) = four;
+      }
     }
   } else {
+    float* buf = s_part + group * n;
+    float ss = 0.f;
     for (int i = me; i < n; i += nth) {
-      const float y = value(i, orow[i], gate_first ? grow[i] : 0.f, skip != nullptr ? qb_to_float<O>(x[(size_t)t * x_stride + c0 + i]) : 0.f);
+      const int h = (c0 + i) / E;
+      float y = orow[i];
+      if (den != nullptr) y = y / den[(size_t)t * H + h];
+      if (skip != nullptr) y = fmaf(skip[h], qb_to_float<O>(xrow[i]), y);
+      if (gate_first) y *= grow[i] / (1.f + expf(-grow[i]));
       ss += y * y;
       buf[i] = y;
     }
-  }
-  if (WARPS == 1) {
-    ss = qb_warp_sum(ss);
-    __syncwarp();
-  } else {
-    ss = qb_block_sum(ss, s_sum);
-  }
-  const float inv = 1.f / sqrtf(ss / (float)n + eps);
-  // every thread finishes the numbers it put there
-  if (vec) {
-    for (int i = me * 4; i < n; i += nth * 4) {
-      const float4 y = *reinterpret_cast<const float4*>(buf + i), gn = *reinterpret_cast<const float4*>(gain + c0 + i);
-      float r[4] = {y.x * inv * gn.x, y.y * inv * gn.y, y.z * inv * gn.z, y.w * inv * gn.w};
-      if (!gate_first) {
-        const float4 gv = *reinterpret_cast<const float4*>(grow + i);
-        r[0] *= 1.f / (1.f + expf(-gv.x));
-        r[1] *= 1.f / (1.f + expf(-gv.y));
-        r[2] *= 1.f / (1.f + expf(-gv.z));
-        r[3] *= 1.f / (1.f + expf(-gv.w));
-      }
-      struct alignas(4 * sizeof(O)) Four { O v[4]; } four;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) four.v[e] = qb_from_float<O>(r[e]);
-      *reinterpret_cast<Four*>(out + (size_t)t * HE + c0 + i) = four;
-    }
-  } else {
-    for (int i = me; i < n; i += nth) {
-      float r = buf[i] * inv * gain[c0 + i];
+    const float inv = root(ss);
+    for (int i = me; i < n; i += nth) {               // every thread finishes the numbers it put there
+      float r = buf[i] * inv * nrow[i];
       if (!gate_first) r *= 1.f / (1.f + expf(-grow[i]));
-      out[(size_t)t * HE + c0 + i] = qb_from_float<O>(r);
+      to[i] = qb_from_float<O>(r);
     }
   }
 }
@@ -1062,25 +1079,35 @@ extern "C" int qb_decay_out(const float* o, const float* den, const void* x, lon
   if (H <= 0 || E <= 0 || parts <= 0 || ((long long)H * E) % parts || (skip != nullptr) != (x != nullptr)) return QB_ERR_BAD_ARG;
   const int n = H * E / parts;
   const bool warp_form = n <= 512;
-  const size_t smem = (size_t)n * (warp_form ? 4 : 1) * sizeof(float);
+  const bool vec = n % 4 == 0 && E % 4 == 0 && gate_stride % 4 == 0 && x_stride % 4 == 0 && n <= 8192 &&
+                   (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out | (uintptr_t)x) & 15) == 0;
+  const int pieces = (n / 4 + (warp_form ? 32 : 256) - 1) / (warp_form ? 32 : 256);
+  const size_t smem = vec ? 0 : (size_t)n * (warp_form ? 4 : 1) * sizeof(float);
   if (smem > 200 * 1024) return QB_ERR_UNSUPPORTED;
-  const int vec = n % 4 == 0 && gate_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out) & 15) == 0;
   const long long units = (long long)T * parts, blocks = warp_form ? (units + 3) / 4 : units;
   if (blocks > 0x7fffffffll) return QB_ERR_UNSUPPORTED;
+#define DS_OUT(WARPS, Q)                                                                                              \
+  do {                                                                                                               \
+    auto kern = decay_out_kernel<O, WARPS, Q>;                                                                        \
+    if (smem > 48 * 1024) {                                                                                           \
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);              \
+      if (e != cudaSuccess) return (int)e;                                                                            \
+    }                                                                                                                 \
+    kern<<<(unsigned)blocks, WARPS == 1 ? 128 : 256, smem, stream>>>(o, den, (const O*)x, x_stride, skip, gate,        \
+                                                                     gate_stride, gain, (O*)out, T, H, E, parts, eps, \
+                                                                     gate_first);                                     \
+  } while (0)
   QB_DISPATCH_DTYPE(out_dtype, O, {
-    if (warp_form) {
-      decay_out_kernel<O, 1><<<(unsigned)blocks, 128, smem, stream>>>(o, den, (const O*)x, x_stride, skip, gate, gate_stride,
-                                                                      gain, (O*)out, T, H, E, parts, eps, gate_first, vec);
-    } else {
-      auto kern = decay_out_kernel<O, 8>;
-      if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return (int)e;
-      }
-      kern<<<(unsigned)blocks, 256, smem, stream>>>(o, den, (const O*)x, x_stride, skip, gate, gate_stride, gain, (O*)out, T, H,
-                                                    E, parts, eps, gate_first, vec);
-    }
+    if (!vec && warp_form) DS_OUT(1, 0);
+    else if (!vec) DS_OUT(8, 0);
+    else if (warp_form && pieces <= 1) DS_OUT(1, 1);
+    else if (warp_form && pieces <= 2) DS_OUT(1, 2);
+    else if (warp_form) DS_OUT(1, 4);
+    else if (pieces <= 2) DS_OUT(8, 2);
+    else if (pieces <= 4) DS_OUT(8, 4);
+    else DS_OUT(8, 8);
   });
+#undef DS_OUT
   QB_LAUNCH_CHECK();
   return 0;
 }

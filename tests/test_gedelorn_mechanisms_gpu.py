@@ -251,7 +251,7 @@ def test_running_maximum(H, cap):
 
 
 # ---- from the recurrence to the output projection ----------------------------------------------------------------
-@pytest.mark.parametrize("H,E,parts", [(4, 12, 4), (3, 10, 1), (2, 96, 2), (6, 20, 3), (8, 128, 1), (5, 7, 5), (16, 64, 2), (2, 300, 4)])
+@pytest.mark.parametrize("H,E,parts", [(4, 12, 4), (3, 10, 1), (2, 96, 2), (6, 20, 3), (8, 128, 1), (5, 7, 5), (16, 64, 2), (2, 300, 4), (32, 128, 1), (8, 640, 2), (4, 2500, 1), (40, 128, 2)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_norm_in_parts_and_gate(H, E, parts, dtype):
     from quanta_b200 import kernels
